@@ -537,6 +537,8 @@ KTK_API int ktk_paged_sv(const void* kv_cache, const int32_t* kv_indices, const 
  *   extend   every listed slot grows by tokens_each tokens (a decode step: 1), taking a new page when it
  *            crosses a page boundary; all or nothing.
  *   release  the slot's pages go back to the pool.
+ *   promise  raises a slot's promise to max_total_tokens (a request whose length is not known at admission);
+ *            KTK_ERR_TOO_LARGE if the pages are not free.
  *   export   for the listed slots, in that order: kv_indices (their pages, concatenated), kv_indptr
  *            [n + 1], kv_last_page_len [n] into host memory of the caller; returns the number of
  *            entries written to kv_indices, or a negative error.
@@ -549,6 +551,7 @@ KTK_API int64_t ktk_pool_free_pages(const ktk_pool* pool);               /* free
 KTK_API int64_t ktk_pool_slot_tokens(const ktk_pool* pool, int32_t slot);  /* -1: slot not in use */
 KTK_API int64_t ktk_pool_slot_pages(const ktk_pool* pool, int32_t slot);
 KTK_API int ktk_pool_admit(ktk_pool* pool, int32_t slot, int64_t n_tokens, int64_t max_total_tokens);
+KTK_API int ktk_pool_promise(ktk_pool* pool, int32_t slot, int64_t max_total_tokens);
 KTK_API int ktk_pool_extend(ktk_pool* pool, const int32_t* slots, int32_t n, int32_t tokens_each);
 KTK_API int ktk_pool_release(ktk_pool* pool, int32_t slot);
 KTK_API int64_t ktk_pool_export(const ktk_pool* pool, const int32_t* slots, int32_t n, int32_t* kv_indices,

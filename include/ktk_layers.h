@@ -1,0 +1,120 @@
+/*
+ * ktk_layers.h -- C ABI of libktk_layers.so: layer mechanisms whose sizes and constants are parameters.
+ *
+ *   residual_norm    residual stream in fp32: add a (normalised) sublayer output, normalise for the next one
+ *   kv_append        keys and values of new tokens into a paged cache with free head sizes
+ *   paged_attention  causal attention over that cache: one or two softmax maps per head over shared values
+ *                    (with two: their weighted difference, unit norm), score softcap, query temperature
+ *   moe_route        router logits, the top experts of each row and their softmax weights, rows per expert
+ *   moe_gemm         the experts' matrix products over the rows routed to them
+ *
+ * Conventions of ktk.h: raw device pointers, cudaStream_t as void*, nothing synchronises or allocates, host-side
+ * argument errors come back as KTK_ERR_*, device-side faults go to a status word and the access is skipped.
+ * The library also carries the page pool and ktk_last_error of ktk.h, so that it can be used alone.
+ *
+ * Row strides are counted in elements and are multiples of 8; columns between the true width and the stride hold
+ * zeros, and every kernel keeps them that way.  `dtype` is that of activations, weights and cache.
+ */
+#ifndef KTK_LAYERS_H_
+#define KTK_LAYERS_H_
+
+#include "ktk.h"
+
+#ifdef __cplusplus
+extern "C" {
+#endif
+
+/* Paged cache of one layer:
+ *   k_pages [num_pages, page_size, kv_heads * maps, dim_stride], v_pages [num_pages, page_size, kv_heads, vdim_stride]
+ * page_size is 16, 32 or 64.  CSR page table as in ktk.h, describing the state AFTER the step's append. */
+typedef struct ktk_paged {
+    const int32_t* kv_indices;
+    const int32_t* kv_indptr;        /* [batch + 1] */
+    const int32_t* kv_last_page_len; /* [batch], in [1, page_size] where a sequence holds pages */
+    int32_t batch;
+    int32_t page_size;
+    int64_t num_pages;
+} ktk_paged;
+
+typedef struct ktk_attn {
+    int32_t heads, kv_heads;         /* query head h reads kv head h / (heads / kv_heads)        */
+    int32_t maps;                    /* 1: softmax(q k) v.  2: a1 - lambda a2 over the same v,
+                                        then / sqrt(mean square + eps), times out_scale          */
+    int32_t dim, vdim;               /* sizes per map and of a value head                        */
+    int32_t dim_stride, vdim_stride; /* the same in memory: multiples of 8, zeros in between     */
+    int32_t dtype;
+    float scale;                     /* score = (q . k) * scale * temperature                    */
+    float softcap;                   /* > 0: score <- softcap * tanh(score / softcap)            */
+    float temp_coef, temp_every;     /* temperature at position p: 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) */
+    float lambda, eps, out_scale;    /* maps = 2 */
+} ktk_attn;
+
+/*
+ * One pass over rows of the fp32 residual stream x [rows, stride]:
+ *   start:   x = embed[token] (tokens and embed given; x is then only written), or x as it lies
+ *   add:     y given: s = sum over `parts` of y[row, part, :];  x += mult * norm(s; post_w, post_b), or
+ *            x += mult * s where post_w is null
+ *   output:  h given: h = norm(x; pre_w, pre_b), in `dtype`
+ * norm(v; w, b) = (v - c) / sqrt(mean((v - c)^2) + eps) * w + b over the first `cols` columns, with c the mean of v
+ * (center != 0) or 0, and b null for none.  Norm weights are fp32 [stride].
+ * zero (nullable): zero_n ints that the launch clears (the expert counters of the router behind it).
+ */
+KTK_API int ktk_residual_norm(const int64_t* tokens, const void* embed, int64_t vocab, float* x, const void* y,
+                              int32_t parts, const float* post_w, const float* post_b, float mult, const float* pre_w,
+                              const float* pre_b, void* h, float eps, int32_t center, int64_t rows, int32_t cols,
+                              int32_t stride, int32_t* zero, int32_t zero_n, int32_t dtype, int32_t* status,
+                              void* stream);
+
+/*
+ * Write K and V of new tokens into their pages.  proj [rows, row_stride] holds each token's keys
+ * (kv_heads * maps * dim_stride) from column k_col and its values (kv_heads * vdim_stride) from column v_col.
+ * new_indptr int32 [batch + 1]: rows of each sequence, its newest tokens; null: one row per sequence.
+ */
+KTK_API int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col, int64_t v_col,
+                          const int32_t* new_indptr, int64_t rows, void* k_pages, void* v_pages,
+                          const ktk_paged* table, const ktk_attn* shape, int32_t* status, void* stream);
+
+/*
+ * Causal attention of new tokens (already in their pages) over their sequence.
+ * q [rows, q_stride]: heads * maps * dim_stride columns, head by head and map by map; o [rows, heads * vdim_stride].
+ * variant: KTK_VARIANT_AUTO, _SIMT (any size, fp32 math), _MMA (bf16, one row per sequence), _UMMA (bf16 on tcgen05).
+ * splits: parts that a sequence's keys are cut into where new_indptr is null (0: policy).
+ */
+KTK_API int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int64_t max_keys);
+KTK_API size_t ktk_paged_attention_workspace(const ktk_attn* shape, int64_t rows, int32_t splits);
+KTK_API int ktk_paged_attention(const void* q, int64_t q_stride, const int32_t* new_indptr, int64_t rows,
+                                int32_t max_new, const void* k_pages, const void* v_pages, const ktk_paged* table,
+                                void* o, void* workspace, size_t workspace_bytes, int32_t splits, int32_t variant,
+                                const ktk_attn* shape, int32_t* status, void* stream);
+
+/* Mixture of experts over rows h [rows, width_stride]. */
+typedef struct ktk_moe {
+    int32_t experts, top;
+    int32_t width, ff;               /* true sizes */
+    int32_t width_stride, ff_stride;
+    int32_t dtype;
+    int32_t reserved;
+} ktk_moe;
+
+/*
+ * logits = W h + b in fp32 (W [experts, width_stride], b fp32); the `top` largest of each row (ties to the lower
+ * expert), weights = softmax over those.  ids / weights [rows, top].  counts [experts] (cleared by the caller):
+ * rows of each expert; bucket [experts, rows]: their row * top + place, in no particular order.
+ */
+KTK_API int ktk_moe_route(const void* h, const void* w, const float* b, int32_t* ids, float* weights, int32_t* counts,
+                          int32_t* bucket, int64_t rows, const ktk_moe* shape, int32_t variant, void* stream);
+
+/*
+ * Expert products.  Rows of expert e take the places [sum of counts before e, + counts[e]) of `act`.
+ *   stage 0: act [rows * top, ff_stride] = silu(G h) * (U h);  w = [experts, 2, ff_stride, width_stride] (G, then U)
+ *   stage 1: y [rows, top, width_stride] = weight * (D act);   w = [experts, width_stride, ff_stride]
+ * variant: KTK_VARIANT_AUTO, _SIMT (fp32 math), _UMMA (bf16 on tcgen05).
+ */
+KTK_API int ktk_moe_gemm(int32_t stage, const void* in, const void* w, void* out, const float* weights,
+                         const int32_t* counts, const int32_t* bucket, int64_t rows, const ktk_moe* shape,
+                         int32_t variant, int32_t* status, void* stream);
+
+#ifdef __cplusplus
+}
+#endif
+#endif

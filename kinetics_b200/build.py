@@ -1,11 +1,13 @@
-"""Build recipe for libktk.so (the C-ABI CUDA library) -- nvcc, sm_100a only.
+"""Build recipe for the C-ABI CUDA libraries -- nvcc, sm_100a only.
 
-Usage: python kinetics_b200/build.py [--force] [--verbose]   (run by path: importing the
-package needs the library this script produces)
+Usage: python kinetics_b200/build.py [--force] [--verbose] [library ...]   (run by path: importing the
+package needs a library this script produces)
 
-Each .cu under csrc/ is compiled to an object under csrc/build/ (skipped when the
-object is newer than the source and every header), then linked into
-kinetics_b200/libktk.so next to this file, so the library travels with the tree.
+  libktk.so         csrc/*.cu: the block top-k paged decode path
+  libktk_layers.so  csrc/layers/*.cu plus the host parts they share with it: layer mechanisms with free sizes
+
+Each source is compiled to an object under csrc/build/<library>/ (skipped when the object is newer than
+the source and every header), then linked next to this file, so the libraries travel with the tree.
 """
 from __future__ import annotations
 
@@ -19,6 +21,12 @@ PKG = Path(__file__).resolve().parent
 CSRC = PKG / "csrc"
 INCLUDE = PKG.parent / "include"
 OUT = PKG / "libktk.so"
+
+#: library -> its sources
+LIBRARIES = {
+    "libktk": lambda: sorted(CSRC.glob("*.cu")),
+    "libktk_layers": lambda: sorted((CSRC / "layers").glob("*.cu")) + [CSRC / "ktk_host.cu", CSRC / "ktk_pool.cu"],
+}
 
 NVCC_FLAGS = [
     "-O3", "-std=c++17", "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo",
@@ -34,12 +42,14 @@ def _nvcc() -> str:
     raise RuntimeError("nvcc not found")
 
 
-def build(force: bool = False, verbose: bool = False) -> Path:
-    sources = sorted(CSRC.glob("*.cu"))
-    headers = sorted(CSRC.glob("*.cuh")) + sorted(INCLUDE.glob("*.h"))
+def build(force: bool = False, verbose: bool = False, library: str = "libktk") -> Path:
+    """Compile what is out of date of one library and link it; returns its path."""
+    sources = LIBRARIES[library]()
+    out = PKG / f"{library}.so"
+    headers = sorted(CSRC.glob("*.cuh")) + sorted((CSRC / "layers").glob("*.cuh")) + sorted(INCLUDE.glob("*.h"))
     newest_header = max(h.stat().st_mtime for h in headers)
-    objdir = CSRC / "build"
-    objdir.mkdir(exist_ok=True)
+    objdir = CSRC / "build" / library
+    objdir.mkdir(parents=True, exist_ok=True)
     nvcc = _nvcc()
 
     def compile_one(src: Path):
@@ -51,7 +61,7 @@ def build(force: bool = False, verbose: bool = False) -> Path:
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"nvcc failed on {src.name}:\n{r.stdout}\n{r.stderr}")
-        return obj, r.stderr
+        return obj, f"{src.name}\n{r.stderr}"
 
     with ThreadPoolExecutor(max_workers=min(8, len(sources))) as ex:
         results = list(ex.map(compile_one, sources))
@@ -61,15 +71,22 @@ def build(force: bool = False, verbose: bool = False) -> Path:
             if log:
                 print(log)
     rebuilt = any(log is not None for _, log in results)
-    if rebuilt or force or not OUT.exists():
-        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", str(OUT),
-               *map(str, objs)]
+    if rebuilt or force or not out.exists() or any(o.stat().st_mtime > out.stat().st_mtime for o in objs):
+        # linked beside its place and moved there, so that a process loading the library never sees half of it
+        part = out.with_suffix(f".{os.getpid()}.part")
+        cmd = [nvcc, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-o", str(part), *map(str, objs)]
         r = subprocess.run(cmd, capture_output=True, text=True)
         if r.returncode != 0:
             raise RuntimeError(f"link failed:\n{r.stdout}\n{r.stderr}")
-    return OUT
+        os.replace(part, out)
+    return out
+
+
+def build_all(force: bool = False, verbose: bool = False):
+    return [build(force, verbose, name) for name in LIBRARIES]
 
 
 if __name__ == "__main__":
-    out = build(force="--force" in sys.argv, verbose="--verbose" in sys.argv or "-v" in sys.argv)
-    print(out)
+    names = [a for a in sys.argv[1:] if not a.startswith("-")] or list(LIBRARIES)
+    for name in names:
+        print(build("--force" in sys.argv, "--verbose" in sys.argv or "-v" in sys.argv, name))

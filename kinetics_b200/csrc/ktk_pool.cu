@@ -101,6 +101,23 @@ extern "C" int ktk_pool_admit(ktk_pool* pool, int32_t slot, int64_t n_tokens, in
     return KTK_OK;
 }
 
+extern "C" int ktk_pool_promise(ktk_pool* pool, int32_t slot, int64_t max_total_tokens) {
+    if (!slot_ok(pool, slot) || pool->tokens[(size_t)slot] < 0 || max_total_tokens < 0) {
+        set_error("ktk_pool_promise: slot %d, %lld tokens at most", slot, (long long)max_total_tokens);
+        return KTK_ERR_ARG;
+    }
+    const int64_t more = pages_for(pool, max_total_tokens) - pool->reserved[(size_t)slot];
+    if (more <= 0) return KTK_OK;
+    if (more > ktk_pool_free_pages(pool)) {
+        set_error("ktk_pool_promise: slot %d needs %lld more pages, %lld are not promised to other sequences", slot,
+                  (long long)more, (long long)ktk_pool_free_pages(pool));
+        return KTK_ERR_TOO_LARGE;
+    }
+    pool->reserved[(size_t)slot] += more;
+    pool->promised += more;
+    return KTK_OK;
+}
+
 extern "C" int ktk_pool_extend(ktk_pool* pool, const int32_t* slots, int32_t n, int32_t tokens_each) {
     if (pool == nullptr || (n > 0 && slots == nullptr) || n < 0 || tokens_each < 0) {
         set_error("ktk_pool_extend: bad arguments");

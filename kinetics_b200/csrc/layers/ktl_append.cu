@@ -1,0 +1,126 @@
+// Keys and values of new tokens -> pages with free head sizes, and the entry point of the attention kernels.
+#include "ktl_common.cuh"
+
+namespace ktk {
+
+// one CTA per row: 16-byte copies of its K and its V row
+template <typename T>
+__global__ void __launch_bounds__(128)
+kv_append_kernel(const T* __restrict__ proj, int64_t row_stride, int64_t k_col, int64_t v_col,
+                 const int32_t* __restrict__ new_indptr, T* __restrict__ k_pages, T* __restrict__ v_pages,
+                 const ktk_paged t, int k_row, int v_row, int32_t* status) {
+    const int64_t r = blockIdx.x;
+    const int b = new_indptr ? sequence_of_row(new_indptr, t.batch, r) : (int)r;
+    const Span s = span_of(t, b);
+    const int pos = new_indptr ? s.total - (new_indptr[b + 1] - (int)r) : s.total - 1;
+    if (s.bad || pos < 0 || pos >= s.total) {
+        if (threadIdx.x == 0) report(status, KTK_STATUS_BAD_TABLE);
+        return;
+    }
+    const int64_t page = t.kv_indices[s.start + pos / t.page_size];
+    if (page < 0 || page >= t.num_pages) {
+        if (threadIdx.x == 0) report(status, KTK_STATUS_BAD_PAGE);
+        return;
+    }
+    const int64_t slot = page * t.page_size + pos % t.page_size;
+    constexpr int kPer = 16 / sizeof(T);
+    const uint4* ks = reinterpret_cast<const uint4*>(proj + r * row_stride + k_col);
+    const uint4* vs = reinterpret_cast<const uint4*>(proj + r * row_stride + v_col);
+    uint4* kd = reinterpret_cast<uint4*>(k_pages + slot * k_row);
+    uint4* vd = reinterpret_cast<uint4*>(v_pages + slot * v_row);
+    for (int i = threadIdx.x; i < k_row / kPer; i += blockDim.x) kd[i] = ks[i];
+    for (int i = threadIdx.x; i < v_row / kPer; i += blockDim.x) vd[i] = vs[i];
+}
+
+template <typename T>
+static int append_launch(const void* proj, int64_t row_stride, int64_t k_col, int64_t v_col, const int32_t* ni,
+                         int64_t rows, void* k, void* v, const ktk_paged& t, int k_row, int v_row, int32_t* status,
+                         cudaStream_t st) {
+    kv_append_kernel<T><<<(unsigned)rows, 128, 0, st>>>((const T*)proj, row_stride, k_col, v_col, ni, (T*)k, (T*)v, t,
+                                                         k_row, v_row, status);
+    KTK_CUDA_TRY(cudaGetLastError(), "ktk_kv_append");
+    return KTK_OK;
+}
+
+}  // namespace ktk
+
+using namespace ktk;
+
+extern "C" int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col, int64_t v_col,
+                             const int32_t* new_indptr, int64_t rows, void* k_pages, void* v_pages,
+                             const ktk_paged* table, const ktk_attn* shape, int32_t* status, void* stream) {
+    const char* who = "ktk_kv_append";
+    const int rc = check_attn(shape, table, who);
+    if (rc != KTK_OK) return rc;
+    if (rows < 0 || rows > 2147483647LL || (!new_indptr && rows != table->batch)) {
+        set_error("%s: %lld rows for %d sequences", who, (long long)rows, table->batch);
+        return KTK_ERR_ARG;
+    }
+    if (rows == 0) return KTK_OK;
+    const int k_row = shape->kv_heads * shape->maps * shape->dim_stride, v_row = shape->kv_heads * shape->vdim_stride;
+    if (!proj || !k_pages || !v_pages || !table->kv_indices || !table->kv_indptr || !table->kv_last_page_len ||
+        row_stride % 8 != 0 || k_col % 8 != 0 || v_col % 8 != 0 || k_col < 0 || v_col < 0 ||
+        k_col + k_row > row_stride || v_col + v_row > row_stride ||
+        (((uintptr_t)proj | (uintptr_t)k_pages | (uintptr_t)v_pages) & 15u) != 0) {
+        set_error("%s: null or misaligned pointer, or columns outside the row", who);
+        return KTK_ERR_ARG;
+    }
+    cudaStream_t st = (cudaStream_t)stream;
+    return shape->dtype == KTK_F32
+               ? append_launch<float>(proj, row_stride, k_col, v_col, new_indptr, rows, k_pages, v_pages, *table, k_row,
+                                      v_row, status, st)
+               : append_launch<__nv_bfloat16>(proj, row_stride, k_col, v_col, new_indptr, rows, k_pages, v_pages,
+                                              *table, k_row, v_row, status, st);
+}
+
+extern "C" int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int64_t max_keys) {
+    return attn_decode_supported(*shape) ? attn_decode_splits(*shape, batch, max_keys) : 1;
+}
+
+extern "C" size_t ktk_paged_attention_workspace(const ktk_attn* shape, int64_t rows, int32_t splits) {
+    return attn_decode_supported(*shape) ? attn_decode_workspace(*shape, rows, splits) : 0;
+}
+
+extern "C" int ktk_paged_attention(const void* q, int64_t q_stride, const int32_t* new_indptr, int64_t rows,
+                                   int32_t max_new, const void* k_pages, const void* v_pages, const ktk_paged* table,
+                                   void* o, void* workspace, size_t workspace_bytes, int32_t splits, int32_t variant,
+                                   const ktk_attn* shape, int32_t* status, void* stream) {
+    const char* who = "ktk_paged_attention";
+    const int rc = check_attn(shape, table, who);
+    if (rc != KTK_OK) return rc;
+    if (rows < 0 || rows > 2147483647LL || (!new_indptr && rows != table->batch) || (new_indptr && max_new < 0)) {
+        set_error("%s: %lld rows for %d sequences, at most %d each", who, (long long)rows, table->batch, max_new);
+        return KTK_ERR_ARG;
+    }
+    if (rows == 0) return KTK_OK;
+    const int q_row = shape->heads * shape->maps * shape->dim_stride;
+    if (!q || !k_pages || !v_pages || !o || !table->kv_indices || !table->kv_indptr || !table->kv_last_page_len ||
+        q_stride < q_row || q_stride % 8 != 0 ||
+        (((uintptr_t)q | (uintptr_t)k_pages | (uintptr_t)v_pages | (uintptr_t)o | (uintptr_t)workspace) & 15u) != 0) {
+        set_error("%s: null or misaligned pointer, or a row stride of %lld", who, (long long)q_stride);
+        return KTK_ERR_ARG;
+    }
+    if (variant < KTK_VARIANT_AUTO || variant > KTK_VARIANT_UMMA) {
+        set_error("%s: unknown variant %d", who, variant);
+        return KTK_ERR_ARG;
+    }
+    AttnParams p{*shape, *table, q, q_stride, new_indptr, rows, max_new, k_pages, v_pages, o, (float*)workspace, splits,
+                 status};
+    const bool can_decode = !new_indptr && attn_decode_supported(*shape);
+    const bool can_umma = new_indptr && attn_umma_supported(*shape);
+    if ((variant == KTK_VARIANT_MMA && !can_decode) || (variant == KTK_VARIANT_UMMA && !can_umma)) {
+        set_error("%s: variant %d is not built for this case", who, variant);
+        return KTK_ERR_UNSUPPORTED;
+    }
+    if (variant != KTK_VARIANT_SIMT && can_umma) return launch_attn_umma(p, (cudaStream_t)stream);
+    if (variant != KTK_VARIANT_SIMT && can_decode) {
+        if (p.splits <= 0) p.splits = attn_decode_splits(*shape, table->batch, 1 << 20);
+        const size_t need = attn_decode_workspace(*shape, rows, p.splits);
+        if (need && (!workspace || workspace_bytes < need)) {
+            set_error("%s: workspace of %zu bytes needed, got %zu", who, need, workspace ? workspace_bytes : (size_t)0);
+            return KTK_ERR_WORKSPACE;
+        }
+        return launch_attn_decode(p, (cudaStream_t)stream);
+    }
+    return launch_attn_simt(p, (cudaStream_t)stream);
+}

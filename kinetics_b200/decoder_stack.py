@@ -106,11 +106,15 @@ class DecoderStack:
         return ops.add_rmsnorm(part, residual, weight, self.eps)
 
     @torch.no_grad()
-    def inference(self, input_ids, position_ids, batch_idx, kv):
+    def inference(self, input_ids, position_ids, batch_idx, kv, rows=None):
+        """fp32 logits [B, S, V]; rows: project only these of the S tokens of one sequence."""
         if self.shard_vocab and self.world > 1:
             raise RuntimeError("inference() returns full logits: build the stack without shard_vocab, or call next_tokens()")
         bsz, seq_len = input_ids.shape
         n = self._hidden(input_ids, position_ids, batch_idx, kv)
+        if rows is not None:
+            n = n[torch.as_tensor(rows, dtype=torch.int64, device=n.device)]
+            bsz, seq_len = 1, len(rows)
         # n is the final RMSNorm of the residual stream (qwen3.py:139)
         logits = torch.mm(n, self.lm_head.t())
         if self.logits_dtype is not None:

@@ -21,7 +21,6 @@ import numpy as np
 import torch
 
 from . import _lib, ops
-from ._lib import check
 from .batch_cache import PAGE, SINK, BatchKVManager
 
 
@@ -37,7 +36,7 @@ class PagePool:
     """Which physical pages each sequence slot owns (``ktk_pool_*``).  Host-only bookkeeping."""
 
     def __init__(self, num_pages: int, max_slots: int, page_size: int = PAGE):
-        self._lib = _lib.load()
+        self._lib = _lib.host()
         self._h = self._lib.ktk_pool_create(num_pages, max_slots, page_size)
         if not self._h:
             raise ValueError(self._lib.ktk_last_error().decode())
@@ -67,17 +66,28 @@ class PagePool:
         rc = self._lib.ktk_pool_admit(self._h, slot, n_tokens, max_total_tokens)
         if rc == _lib.KTK_ERR_TOO_LARGE:
             raise PoolExhausted(self._lib.ktk_last_error().decode())
-        check(rc)
+        self._check(rc)
+
+    def promise(self, slot: int, max_total_tokens: int) -> None:
+        """Raise the slot's promise (a request whose length was not known at admission)."""
+        rc = self._lib.ktk_pool_promise(self._h, slot, max_total_tokens)
+        if rc == _lib.KTK_ERR_TOO_LARGE:
+            raise PoolExhausted(self._lib.ktk_last_error().decode())
+        self._check(rc)
+
+    def _check(self, rc: int) -> None:
+        if rc != 0:
+            raise _lib.KtkError(rc, self._lib.ktk_last_error().decode())
 
     def extend(self, slots: Sequence[int], tokens_each: int = 1) -> None:
         arr = (ctypes.c_int32 * len(slots))(*slots)
         rc = self._lib.ktk_pool_extend(self._h, arr, len(slots), tokens_each)
         if rc == _lib.KTK_ERR_TOO_LARGE:
             raise PoolExhausted(self._lib.ktk_last_error().decode())
-        check(rc)
+        self._check(rc)
 
     def release(self, slot: int) -> None:
-        check(self._lib.ktk_pool_release(self._h, slot))
+        self._check(self._lib.ktk_pool_release(self._h, slot))
 
     def export(self, slots: Sequence[int], pin: bool = False):
         """(kv_indices, kv_indptr, kv_last_page_len) as int32 CPU tensors for the slots, in that order."""
@@ -90,7 +100,7 @@ class PagePool:
         total = self._lib.ktk_pool_export(self._h, arr, n, ctypes.c_void_p(indices.data_ptr()), cap,
                                           ctypes.c_void_p(indptr.data_ptr()), ctypes.c_void_p(last.data_ptr()))
         if total < 0:
-            check(int(total))
+            self._check(int(total))
         return indices[:total], indptr, last[:n]
 
 
@@ -106,7 +116,7 @@ class PagePool:
         total = self._lib.ktk_pool_export(self._h, arr, n, ctypes.c_void_p(indices.data_ptr()), indices.numel(),
                                           ctypes.c_void_p(indptr.data_ptr()), ctypes.c_void_p(last.data_ptr()))
         if total < 0:
-            check(int(total))
+            self._check(int(total))
         return int(total)
 
 
@@ -114,46 +124,21 @@ class PagePool:
 # KV manager backed by the pool
 # --------------------------------------------------------------------------------------
 
-def _pool_tokens(length: int) -> int:
-    """Tokens the pool has to hold for a sequence of `length` tokens: the sink page (4 tokens) takes a
-    whole page, the pages behind it are ordinary 16-token pages (see batch_cache.py)."""
-    if length <= 0:
-        return 0
-    return PAGE + max(length - SINK, 0)
+class PooledTable:
+    """Slots, their pages and the page table of a step: what the KV managers on a ``PagePool`` share.
 
-
-class PooledKVManager(BatchKVManager):
-    """``BatchKVManager`` whose pages come from a ``PagePool`` shared by all slots.
-
-    Same attention surface (``compute_attention`` / ``decode`` / ``prefill_or_append`` /
-    ``clear_cache``); in addition ``admit(slot, prompt_len, max_total_len)`` has to be called before a
-    slot is first written (the engine does), and ``begin_step(slots)`` may be called with the active
-    slots as a host list to spare the manager a device-to-host read of ``batch_idx``.
+    The host knows every slot's length (``_host_len`` per layer), so no step reads one back.  With ``sink`` > 0 the
+    first page of a sequence holds only its first ``sink`` tokens (see batch_cache.py).  ``admit(slot, prompt_len,
+    max_total_len)`` has to be called before a slot is first written (the engine does), and ``begin_step(slots)``
+    may be called with the active slots as a host list to spare a device-to-host read of ``batch_idx``.
     """
 
-    def __init__(self, config, max_batch_size: int, max_seq_len: int, device, dtype, num_pages: int,
-                 alias_layers: bool = False, **kwargs):
-        """`alias_layers`: every layer reads and writes ONE physical pool and one summary table (a benchmark
-        device for models whose caches would not fit: the traffic per layer is real, the contents are not)."""
+    sink = 0
+    page_size = PAGE
+
+    def _init_table(self, num_pages: int) -> None:
         self._num_pool_pages = int(num_pages)
-        self._alias = bool(alias_layers)
-        super().__init__(config, max_batch_size, max_seq_len, device, dtype, **kwargs)
-
-    def _alloc_summaries(self):
-        if not self._alias:
-            return super()._alloc_summaries()
-        one = torch.zeros(self.max_batch_size, self.num_key_value_heads, self.pages_per_slot, self.head_dim,
-                          device=self.device, dtype=self.dtype)
-        return [one] * self.num_layers
-
-    # BatchKVManager allocates pages_per_slot * max_batch pages per layer; here the pool decides
-    def _alloc_pages(self):
-        total = self._num_pool_pages
-        self.pool = PagePool(total, self.max_batch_size, PAGE)
-        def pages():
-            return torch.zeros(total, 2, PAGE, self.num_key_value_heads, self.head_dim, device=self.device,
-                               dtype=self.dtype)
-        self.kv_pages = [pages()] * self.num_layers if self._alias else [pages() for _ in range(self.num_layers)]
+        self.pool = PagePool(self._num_pool_pages, self.max_batch_size, self.page_size)
         self.kv_indices = None
         self._host_len = np.zeros((self.num_layers, self.max_batch_size), dtype=np.int64)
         self._active: Optional[List[int]] = None
@@ -164,21 +149,42 @@ class PooledKVManager(BatchKVManager):
         self._copies_done = None         # event behind the last step's table copies
         self._static = None              # static device buffers + pinned mirrors of that table
 
+    def _pool_tokens(self, length):
+        """Tokens the pool has to hold for a sequence of `length` (an int or an array of them): a sink takes a
+        whole page, the pages behind it are ordinary ones."""
+        if self.sink == 0:
+            return length
+        return np.where(np.asarray(length) > 0, self.page_size + np.maximum(np.asarray(length) - self.sink, 0), 0)
+
+    def _last_fill(self, lengths):
+        """Tokens in the last page of sequences of these lengths (an array)."""
+        n = np.asarray(lengths)
+        behind = (n - self.sink - 1) % self.page_size + 1
+        return np.where(n <= self.sink, n, behind)
+
+    def _view(self, slots, order=None):
+        """How the pages split for the kernels of this manager (a PageView, or None)."""
+        return None
+
     # ---- admission / retirement
     def can_admit(self, max_total_len: int) -> bool:
-        return self.pool.can_admit(_pool_tokens(max_total_len))
+        return self.pool.can_admit(int(self._pool_tokens(max_total_len)))
 
     def admit(self, slot: int, prompt_len: int, max_total_len: int) -> None:
         if max_total_len > self.max_length:
             raise ValueError(f"{max_total_len} tokens exceed max_seq_len {self.max_length}")
-        self.pool.admit(slot, 0, _pool_tokens(max_total_len))
+        self.pool.admit(slot, 0, int(self._pool_tokens(max_total_len)))
 
-    def clear_cache(self, batch_idx: int):
-        super().clear_cache(batch_idx)
-        for i in range(self.num_layers):
-            self._host_len[i][batch_idx] = 0
-        if self.pool.tokens(batch_idx) >= 0:
-            self.pool.release(batch_idx)
+    def promise(self, slot: int, max_total_len: int) -> None:
+        """Raise what was promised at admission (a request that turns out longer)."""
+        if max_total_len > self.max_length:
+            raise ValueError(f"{max_total_len} tokens exceed max_seq_len {self.max_length}")
+        self.pool.promise(slot, int(self._pool_tokens(max_total_len)))
+
+    def _release_slot(self, slot: int) -> None:
+        self._host_len[:, slot] = 0
+        if self.pool.tokens(slot) >= 0:
+            self.pool.release(slot)
         self._table_key = None
 
     def begin_step(self, slots: Sequence[int]) -> None:
@@ -213,12 +219,11 @@ class PooledKVManager(BatchKVManager):
         self.wait_for_table_copies()
         idx = np.asarray(slots, dtype=np.int64)
         lengths = self._host_len[0, idx] + 1
-        pool_tokens = lambda ln: np.where(ln > 0, PAGE + np.maximum(ln - SINK, 0), 0)
-        grow = idx[pool_tokens(lengths) > pool_tokens(lengths - 1)]
+        grow = idx[self._pool_tokens(lengths) > self._pool_tokens(lengths - 1)]
         if grow.size:
             self.pool.extend(grow.tolist(), 1)
         total = self.pool.export_into(slots, st["h_indices"], st["h_indptr"], st["h_last"])
-        st["h_last"].numpy()[:n] = np.where(lengths <= SINK, lengths, (lengths - SINK - 1) % PAGE + 1)
+        st["h_last"].numpy()[:n] = self._last_fill(lengths)
         st["h_slot"].numpy()[:n] = idx
         # rows of the batch from the longest to the shortest: the selection kernel's CTAs share them evenly
         st["h_order"].numpy()[:n] = np.argsort(-lengths, kind="stable")
@@ -230,7 +235,7 @@ class PooledKVManager(BatchKVManager):
         if self._copies_done is None:
             self._copies_done = torch.cuda.Event()
         self._copies_done.record()
-        view = ops.PageView(SINK, self.local, None, st["d_slot"][:n], st["d_order"][:n])
+        view = self._view(st["d_slot"][:n], st["d_order"][:n])
         self._step_table = (st["d_indices"], st["d_indptr"][:n + 1], st["d_last"][:n], view)
         self._step_offsets_advanced = False
         self.kv_indices = st["d_indices"]
@@ -238,34 +243,11 @@ class PooledKVManager(BatchKVManager):
         self._active = slots
         self.table_bytes = 4 * (total + 4 * n + 1)
         # pages the step opened (a promise made at admission may already have reserved them)
-        self.pages_opened = int(np.count_nonzero((lengths - SINK - 1) % PAGE == 0)) if n else 0
+        self.pages_opened = int(np.count_nonzero((lengths - self.sink - 1) % self.page_size == 0)) if n else 0
 
     def end_step(self) -> None:
         self._step_table = None
         self._table_key = None
-
-    def assume_filled(self, lengths: dict, headroom: int = 0) -> None:
-        """Benchmark set-up: slot -> number of tokens its pages are taken to hold already (the page contents
-        are whatever the pool memory holds).  Admits the slots with a promise of `headroom` more tokens, grows
-        them to that length, sets the lengths of every layer and rebuilds the page summaries from the pages."""
-        slots = sorted(lengths)
-        for s in slots:
-            self.pool.admit(s, _pool_tokens(lengths[s]), _pool_tokens(min(lengths[s] + headroom, self.max_length)))
-        lens_t = torch.zeros(self.max_batch_size, dtype=torch.int32)
-        for s in slots:
-            lens_t[s] = lengths[s]
-        for layer in range(self.num_layers):
-            self.kv_offset[layer].copy_(lens_t)
-            for s in slots:
-                self._host_len[layer][s] = lengths[s]
-        indices, indptr, _ = self.pool.export(slots)
-        last = torch.tensor([n if n <= SINK else (n - SINK - 1) % PAGE + 1 for n in (lengths[s] for s in slots)],
-                            dtype=torch.int32)
-        dev = self.device
-        view = ops.PageView(SINK, self.local, None, torch.tensor(slots, dtype=torch.int32, device=dev))
-        for layer in range(1 if self._alias else self.num_layers):
-            ops.build_summaries(self.kv_pages[layer], self.summaries[layer], indices.to(dev), indptr.to(dev),
-                                last.to(dev), status=self.status, view=view)
 
     # ---- page table of the active rows
     def _slots_of(self, batch_idx: torch.Tensor) -> List[int]:
@@ -282,19 +264,84 @@ class PooledKVManager(BatchKVManager):
             have = self.pool.tokens(s)
             if have < 0:
                 raise RuntimeError(f"slot {s} was not admitted to the page pool")
-            d = _pool_tokens(n) - have
+            d = int(self._pool_tokens(n)) - have
             if d > 0:
                 grow.setdefault(d, []).append(s)
         for d, ss in grow.items():
             self.pool.extend(ss, d)
         indices, indptr, _ = self.pool.export(slots, pin=True)
-        last = torch.tensor([n if n <= SINK else (n - SINK - 1) % PAGE + 1 for n in lengths], dtype=torch.int32)
+        last = torch.from_numpy(self._last_fill(lengths).astype(np.int32))
         slot_t = torch.tensor(slots, dtype=torch.int32)
         dev = self.device
         val = (indices.to(dev, non_blocking=True), indptr.to(dev, non_blocking=True),
-               last.to(dev, non_blocking=True), ops.PageView(SINK, self.local, None, slot_t.to(dev)))
+               last.to(dev, non_blocking=True), self._view(slot_t.to(dev)))
         self._table_key, self._table_val = key, val
         return val
+
+
+class PooledKVManager(PooledTable, BatchKVManager):
+    """``BatchKVManager`` whose pages come from a ``PagePool`` shared by all slots.
+
+    Same attention surface (``compute_attention`` / ``decode`` / ``prefill_or_append`` /
+    ``clear_cache``), and the admission and step calls of ``PooledTable``.
+    """
+
+    sink = SINK
+
+    def __init__(self, config, max_batch_size: int, max_seq_len: int, device, dtype, num_pages: int,
+                 alias_layers: bool = False, **kwargs):
+        """`alias_layers`: every layer reads and writes ONE physical pool and one summary table (a benchmark
+        device for models whose caches would not fit: the traffic per layer is real, the contents are not)."""
+        self._num_pool_pages = int(num_pages)
+        self._alias = bool(alias_layers)
+        super().__init__(config, max_batch_size, max_seq_len, device, dtype, **kwargs)
+
+    def _alloc_summaries(self):
+        if not self._alias:
+            return super()._alloc_summaries()
+        one = torch.zeros(self.max_batch_size, self.num_key_value_heads, self.pages_per_slot, self.head_dim,
+                          device=self.device, dtype=self.dtype)
+        return [one] * self.num_layers
+
+    # BatchKVManager allocates pages_per_slot * max_batch pages per layer; here the pool decides
+    def _alloc_pages(self):
+        total = self._num_pool_pages
+        self._init_table(total)
+
+        def pages():
+            return torch.zeros(total, 2, PAGE, self.num_key_value_heads, self.head_dim, device=self.device,
+                               dtype=self.dtype)
+        self.kv_pages = [pages()] * self.num_layers if self._alias else [pages() for _ in range(self.num_layers)]
+
+    def _view(self, slots, order=None):
+        return ops.PageView(SINK, self.local, None, slots, order)
+
+    def clear_cache(self, batch_idx: int):
+        super().clear_cache(batch_idx)
+        self._release_slot(batch_idx)
+
+    def assume_filled(self, lengths: dict, headroom: int = 0) -> None:
+        """Benchmark set-up: slot -> number of tokens its pages are taken to hold already (the page contents
+        are whatever the pool memory holds).  Admits the slots with a promise of `headroom` more tokens, grows
+        them to that length, sets the lengths of every layer and rebuilds the page summaries from the pages."""
+        slots = sorted(lengths)
+        for s in slots:
+            self.pool.admit(s, int(self._pool_tokens(lengths[s])),
+                            int(self._pool_tokens(min(lengths[s] + headroom, self.max_length))))
+        lens_t = torch.zeros(self.max_batch_size, dtype=torch.int32)
+        for s in slots:
+            lens_t[s] = lengths[s]
+        for layer in range(self.num_layers):
+            self.kv_offset[layer].copy_(lens_t)
+            for s in slots:
+                self._host_len[layer][s] = lengths[s]
+        indices, indptr, _ = self.pool.export(slots)
+        last = torch.from_numpy(self._last_fill([lengths[s] for s in slots]).astype(np.int32))
+        dev = self.device
+        view = ops.PageView(SINK, self.local, None, torch.tensor(slots, dtype=torch.int32, device=dev))
+        for layer in range(1 if self._alias else self.num_layers):
+            ops.build_summaries(self.kv_pages[layer], self.summaries[layer], indices.to(dev), indptr.to(dev),
+                                last.to(dev), status=self.status, view=view)
 
     def _table(self, batch_idx: torch.Tensor, lengths: torch.Tensor):
         raise RuntimeError("PooledKVManager builds its page table from host lengths (_table_for)")
@@ -403,8 +450,11 @@ class Engine:
     def __init__(self, model, kv, max_seq_len: int, device, top_p: float = 1.0, temperature: float = 0.0,
                  top_k: int = 0, eos: Sequence[int] = (151643, 151645), repeat_check: bool = True,
                  repeat_check_window: int = 1024, repeat_block_size: int = 64, seed: Optional[int] = None,
-                 preprocess: Optional[Callable] = None, postprocess: Optional[Callable] = None):
+                 preprocess: Optional[Callable] = None, postprocess: Optional[Callable] = None,
+                 prefill_chunk: int = 0):
+        """prefill_chunk: a prompt runs in portions of at most this many tokens (0: whole)."""
         self.model, self.kv = model, kv
+        self.prefill_chunk = int(prefill_chunk)
         self.device = torch.device(device)
         self.max_seq_len = max_seq_len
         self.max_batch_size = kv.max_batch_size
@@ -442,17 +492,59 @@ class Engine:
             raise ValueError(f"prompt of {prompt_len} tokens + {max_new_tokens} new ones exceed max_seq_len")
         return self.kv.can_admit(total) if hasattr(self.kv, "can_admit") else True
 
+    def open_slot(self, slot: int, max_total_tokens: int = 0) -> None:
+        """Take a free slot for a request whose tokens come with `extend`; max_total_tokens: pages to promise it now
+        (`extend` asks the pool for more where that is not enough)."""
+        if self.slots_occupy_status[slot]:
+            raise ValueError(f"slot {slot} is occupied")
+        if hasattr(self.kv, "admit"):
+            self.kv.admit(slot, 0, max_total_tokens)
+        self.slots_occupy_status[slot] = True
+
+    def extend(self, slot: int, tokens, want: Sequence[int] = ()) -> Optional[torch.Tensor]:
+        """Run the next tokens of an open slot on top of what its cache holds; returns the logits [len(want), V] at
+        the wanted places among them (None where nothing is wanted).  Nothing is sampled."""
+        if not self.slots_occupy_status[slot]:
+            raise ValueError(f"slot {slot} is not open")
+        ids = torch.as_tensor(tokens, dtype=torch.long).reshape(1, -1).to(self.device)
+        n, held = ids.shape[1], self._offsets_host[slot]
+        if held + n > self.max_seq_len:
+            raise ValueError(f"{held} + {n} tokens exceed max_seq_len {self.max_seq_len}")
+        if hasattr(self.kv, "promise"):
+            self.kv.promise(slot, held + n)
+        self.slots_tokens[slot, held:held + n].copy_(ids[0])
+        logits = self._run_portion(slot, ids, held, list(want))
+        self.slots_offsets[slot] = held + n
+        self._offsets_host[slot] = held + n
+        return logits
+
+    def _run_portion(self, slot: int, ids: torch.Tensor, start: int, rows: Optional[List[int]]):
+        """One forward over ids [1, n] of the slot's sequence, positions start ..; logits of `rows`, [len, V]."""
+        n = ids.shape[1]
+        position_ids = torch.arange(start, start + n, dtype=torch.long, device=self.device).unsqueeze(0)
+        batch_idx = torch.tensor([slot], device=self.device)
+        if hasattr(self.kv, "begin_step"):
+            self.kv.begin_step([slot])
+        logits = self.model.inference(ids, position_ids, batch_idx, self.kv, rows=rows)
+        return logits[0] if rows else None
+
     def prefill(self, slot: int, input_ids: torch.Tensor, max_new_tokens: int) -> None:
         seq_len = input_ids.shape[1]
         if hasattr(self.kv, "admit"):
             self.kv.admit(slot, seq_len, seq_len + max_new_tokens)
         input_ids = input_ids.to(self.device)
-        position_ids = torch.arange(seq_len, dtype=torch.long, device=self.device).unsqueeze(0)
         self.slots_tokens[slot, :seq_len].copy_(input_ids[0])
         self.slots_offsets[slot] = seq_len
         self.slots_prompt_len[slot] = seq_len
         self._offsets_host[slot] = self._prompt_host[slot] = seq_len
         self.slots_occupy_status[slot] = True
+        start = 0
+        if self.prefill_chunk > 0:
+            while seq_len - start > self.prefill_chunk:         # all portions but the last: nothing is projected
+                self._run_portion(slot, input_ids[:, start:start + self.prefill_chunk], start, [])
+                start += self.prefill_chunk
+        input_ids = input_ids[:, start:]
+        position_ids = torch.arange(start, seq_len, dtype=torch.long, device=self.device).unsqueeze(0)
         batch_idx = torch.tensor([slot], device=self.device)
         if hasattr(self.kv, "begin_step"):
             self.kv.begin_step([slot])
