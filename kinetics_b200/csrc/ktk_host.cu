@@ -76,9 +76,8 @@ typedef CUresult (*encode_tiled_fn)(CUtensorMap*, CUtensorMapDataType, cuuint32_
                                     CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion,
                                     CUtensorMapFloatOOBfill);
 
-int make_tensor_map_3d(CUtensorMap* out, const void* base, CUtensorMapDataType dt, const uint64_t dims[3],
-                       const uint64_t strides_bytes[2], const uint32_t box[3], CUtensorMapSwizzle swizzle,
-                       const char* who) {
+int make_tensor_map(CUtensorMap* out, const void* base, CUtensorMapDataType dt, int rank, const uint64_t* dims,
+                    const uint64_t* strides_bytes, const uint32_t* box, CUtensorMapSwizzle swizzle, const char* who) {
     static encode_tiled_fn encode = nullptr;
     if (encode == nullptr) {
         void* fn = nullptr;
@@ -91,18 +90,26 @@ int make_tensor_map_3d(CUtensorMap* out, const void* base, CUtensorMapDataType d
         }
         encode = (encode_tiled_fn)fn;
     }
-    cuuint64_t gdim[3] = {dims[0], dims[1], dims[2]};
-    cuuint64_t gstr[2] = {strides_bytes[0], strides_bytes[1]};
-    cuuint32_t bx[3] = {box[0], box[1], box[2]};
-    cuuint32_t es[3] = {1, 1, 1};
-    CUresult r = encode(out, dt, 3, const_cast<void*>(base), gdim, gstr, bx, es, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                        swizzle, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+    cuuint64_t gdim[5] = {1, 1, 1, 1, 1}, gstr[4] = {0, 0, 0, 0};
+    cuuint32_t bx[5] = {1, 1, 1, 1, 1}, es[5] = {1, 1, 1, 1, 1};
+    if (rank < 1 || rank > 5) { set_error("%s: tensor map of rank %d", who, rank); return KTK_ERR_ARG; }
+    for (int i = 0; i < rank; ++i) { gdim[i] = dims[i]; bx[i] = box[i]; }
+    for (int i = 0; i + 1 < rank; ++i) gstr[i] = strides_bytes[i];
+    CUresult r = encode(out, dt, (cuuint32_t)rank, const_cast<void*>(base), gdim, gstr, bx, es,
+                        CU_TENSOR_MAP_INTERLEAVE_NONE, swizzle, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
+                        CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     if (r != CUDA_SUCCESS) {
         set_error("%s: cuTensorMapEncodeTiled failed with %d (base %p, dims %llu x %llu x %llu)", who, (int)r,
-                  base, (unsigned long long)dims[0], (unsigned long long)dims[1], (unsigned long long)dims[2]);
+                  base, (unsigned long long)gdim[0], (unsigned long long)gdim[1], (unsigned long long)gdim[2]);
         return KTK_ERR_CUDA;
     }
     return KTK_OK;
+}
+
+int make_tensor_map_3d(CUtensorMap* out, const void* base, CUtensorMapDataType dt, const uint64_t dims[3],
+                       const uint64_t strides_bytes[2], const uint32_t box[3], CUtensorMapSwizzle swizzle,
+                       const char* who) {
+    return make_tensor_map(out, base, dt, 3, dims, strides_bytes, box, swizzle, who);
 }
 
 }  // namespace ktk

@@ -113,6 +113,10 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
     return *reinterpret_cast<const uint32_t*>(&v);
 }
 
+// Host: build a tiled tensor map.  dims / box innermost first; strides in bytes for dims 1 ...
+int make_tensor_map(CUtensorMap* out, const void* base, CUtensorMapDataType dt, int rank, const uint64_t* dims,
+                    const uint64_t* strides_bytes, const uint32_t* box, CUtensorMapSwizzle swizzle, const char* who);
+
 // Host: build a 3-D tiled tensor map.  dims/strides innermost first; strides in bytes for dims 1..2.
 int make_tensor_map_3d(CUtensorMap* out, const void* base, CUtensorMapDataType dt, const uint64_t dims[3],
                        const uint64_t strides_bytes[2], const uint32_t box[3], CUtensorMapSwizzle swizzle,

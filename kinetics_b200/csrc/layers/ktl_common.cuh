@@ -79,6 +79,7 @@ int launch_attn_simt(const AttnParams& p, cudaStream_t st);
 bool attn_decode_supported(const ktk_attn& a);
 int32_t attn_decode_splits(const ktk_attn& a, int batch, int64_t max_keys);
 size_t attn_decode_workspace(const ktk_attn& a, int64_t rows, int splits);
+int make_cache_maps(const AttnParams& p, struct CUtensorMap_st* k_map, struct CUtensorMap_st* v_map, unsigned box_rows, const char* who);
 int launch_attn_decode(const AttnParams& p, cudaStream_t st);
 bool attn_umma_supported(const ktk_attn& a);
 int launch_attn_umma(const AttnParams& p, cudaStream_t st);
