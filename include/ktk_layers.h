@@ -106,7 +106,8 @@ KTK_API int ktk_moe_route(const void* h, const void* w, const float* b, int32_t*
 
 /*
  * Expert products.  Rows of expert e take the places [sum of counts before e, + counts[e]) of `act`.
- *   stage 0: act [rows * top, ff_stride] = silu(G h) * (U h);  w = [experts, 2, ff_stride, width_stride] (G, then U)
+ *   stage 0: act [rows * top, ff_stride] = silu(G h) * (U h);  w = [experts, ff_stride, 2, width_stride] (a row of G, then
+ *            the row of U of the same inner column)
  *   stage 1: y [rows, top, width_stride] = weight * (D act);   w = [experts, width_stride, ff_stride]
  * variant: KTK_VARIANT_AUTO, _SIMT (fp32 math), _UMMA (bf16 on tcgen05).
  */

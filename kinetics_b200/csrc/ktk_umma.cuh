@@ -140,13 +140,4 @@ __device__ __forceinline__ void tmem_alloc(uint32_t* base_smem, uint32_t cols) {
 __device__ __forceinline__ void tmem_free(uint32_t base, uint32_t cols) {
     asm volatile("tcgen05.dealloc.cta_group::1.sync.aligned.b32 %0, %1;" ::"r"(base), "r"(cols) : "memory");
 }
-// Four rows of a 2-D tensor (box: 64 elements x 1 row) -> 4 x 128 bytes of shared memory, completion counted on `bar`.
-__device__ __forceinline__ void tma_gather4(void* dst, const CUtensorMap* map, uint64_t* bar, int x, const int (&r)[4]) {
-    asm volatile(
-        "cp.async.bulk.tensor.2d.shared::cta.global.tile::gather4.mbarrier::complete_tx::bytes "
-        "[%0], [%1, {%3, %4, %5, %6, %7}], [%2];"
-        ::"r"(smem_u32(dst)), "l"(map), "r"(smem_u32(bar)), "r"(x), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3])
-        : "memory");
-}
-
 }  // namespace ktk

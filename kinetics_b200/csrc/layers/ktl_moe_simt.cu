@@ -49,7 +49,7 @@ __global__ void __launch_bounds__(kMsThreads) moe_simt_kernel(const MoeParams p)
                 sa[kk][rr] = s >= 0 && k0 + kk < K ? to_f32(((const T*)p.in)[s * K + k0 + kk]) : 0.0f;
 #pragma unroll
                 for (int g = 0; g < (STAGE == 0 ? 2 : 1); ++g) {
-                    const int64_t wr = (STAGE == 0 ? (int64_t)e * 2 + g : (int64_t)e) * N + n0 + rr;
+                    const int64_t wr = STAGE == 0 ? ((int64_t)e * N + n0 + rr) * 2 + g : (int64_t)e * N + n0 + rr;
                     sb[g][kk][rr] = n0 + rr < N && k0 + kk < K ? to_f32(((const T*)p.w)[wr * K + k0 + kk]) : 0.0f;
                 }
             }

@@ -97,30 +97,31 @@ class Gifetar:
         self.eps, self.mult = config.norm_eps, config.residual_mult
         self.status = ops.new_status(self.device)
         W, C, S = weights, config.width, self.stride
+        zeros = lambda *shape: torch.zeros(*shape, dtype=dtype, device=self.device)
 
         def heads(name, groups, size, cols=C):
             """[groups * size, cols] -> [groups * pad8(size), stride], zeros in the padding."""
             t = W[name]
             if tuple(t.shape) != (groups * size, cols):
                 raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {(groups * size, cols)}")
-            out = torch.zeros(groups, pad8(size), pad8(cols), dtype=dtype)
+            out = zeros(groups, pad8(size), pad8(cols))
             out[:, :size, :cols] = t.view(groups, size, cols)
-            return out.view(groups * pad8(size), pad8(cols)).to(self.device)
+            return out.view(groups * pad8(size), pad8(cols))
 
         def vector(name, groups, size, to=torch.float32):
             t = W[name]
             if t.numel() != groups * size:
                 raise ValueError(f"{name}: {t.numel()} values, expected {groups * size}")
-            out = torch.zeros(groups, pad8(size), dtype=to)
+            out = torch.zeros(groups, pad8(size), dtype=to, device=self.device)
             out[:, :size] = t.view(groups, size)
-            return out.view(-1).to(self.device)
+            return out.view(-1)
 
         norm = lambda name: (vector(name, 1, C), vector(name + ".b", 1, C))
         table = W["embed"]
         if tuple(table.shape) != (config.vocab, C):
             raise ValueError(f"embed: shape {tuple(table.shape)}, expected {(config.vocab, C)}")
-        self.embed = torch.zeros(config.vocab, S, dtype=dtype, device=self.device)
-        self.embed[:, :C] = table.to(self.device, dtype)
+        self.embed = zeros(config.vocab, S)
+        self.embed[:, :C] = table
         self.final_norm = norm("final.norm")
         self.layers, self.attention_specs = [], []
         for i, l in enumerate(config.layers):
@@ -132,7 +133,7 @@ class Gifetar:
             o = W[mx + "o"]
             if tuple(o.shape) != (C, l.heads * l.vdim):
                 raise ValueError(f"{mx}o: shape {tuple(o.shape)}, expected {(C, l.heads * l.vdim)}")
-            o_pad = torch.zeros(S, l.heads, spec.vdim_stride, dtype=dtype)
+            o_pad = zeros(S, l.heads, spec.vdim_stride)
             o_pad[:C, :, :l.vdim] = o.view(C, l.heads, l.vdim)
             layer = dict(
                 norm1=norm(p + "norm1"), norm1b=norm(p + "norm1b"), spec=spec, moe=l.moe(C),
@@ -140,20 +141,18 @@ class Gifetar:
                                 heads(mx + "v", l.kv_heads, l.vdim))),
                 bqkv=torch.cat((vector(mx + "q.b", H2, l.dim, dtype), vector(mx + "k.b", G2, l.dim, dtype),
                                 vector(mx + "v.b", l.kv_heads, l.vdim, dtype))),
-                wo=o_pad.view(S, l.heads * spec.vdim_stride).to(self.device))
+                wo=o_pad.view(S, l.heads * spec.vdim_stride))
             if layer["moe"] is not None:
                 f, ml = l.ff, p + "mlp."
-                gate_up = torch.zeros(l.experts, 2, pad8(f), S, dtype=dtype)
-                down = torch.zeros(l.experts, S, pad8(f), dtype=dtype)
+                gate_up, down = zeros(l.experts, pad8(f), 2, S), zeros(l.experts, S, pad8(f))
                 for e in range(l.experts):
-                    gate_up[e, 0, :f, :C] = W[f"{ml}e{e}.gate"]
-                    gate_up[e, 1, :f, :C] = W[f"{ml}e{e}.up"]
+                    gate_up[e, :f, 0, :C] = W[f"{ml}e{e}.gate"]
+                    gate_up[e, :f, 1, :C] = W[f"{ml}e{e}.up"]
                     down[e, :C, :f] = W[f"{ml}e{e}.down"]
-                router = torch.zeros(l.experts, S, dtype=dtype)
+                router = zeros(l.experts, S)
                 router[:, :C] = W[ml + "router"]
-                layer.update(norm2=norm(p + "norm2"), norm2b=norm(p + "norm2b"), router=router.to(self.device),
-                             router_b=W[ml + "router.b"].float().to(self.device), gate_up=gate_up.to(self.device),
-                             down=down.to(self.device),
+                layer.update(norm2=norm(p + "norm2"), norm2b=norm(p + "norm2b"), router=router,
+                             router_b=W[ml + "router.b"].float().to(self.device), gate_up=gate_up, down=down,
                              counts=torch.zeros(l.experts, dtype=torch.int32, device=self.device))
             self.layers.append(layer)
             self.attention_specs.append(spec)

@@ -196,7 +196,7 @@ class Routing:
         self.bucket = torch.empty(spec.experts, rows, dtype=torch.int32, device=device)
 
 
-def moe_route(h, w, b, spec: MoeSpec, counts=None) -> Routing:
+def moe_route(h, w, b, spec: MoeSpec, counts=None, variant: int = VARIANT_AUTO) -> Routing:
     """Router of rows h [rows, pad8(width)]: w [experts, pad8(width)] in the dtype of h, b fp32 [experts].  counts:
     a cleared int32 [experts] tensor to count into (None: a new one)."""
     _cuda(h, w, b, counts)
@@ -205,7 +205,7 @@ def moe_route(h, w, b, spec: MoeSpec, counts=None) -> Routing:
     r = Routing(spec, h.shape[0], h.device, counts)
     m = spec.c(_dtype_code(h))
     check_layers(_lib.load_layers().ktk_moe_route(_ptr(h), _ptr(w), _ptr(b), _ptr(r.ids), _ptr(r.weights),
-                                                  _ptr(r.counts), _ptr(r.bucket), h.shape[0], ctypes.byref(m), 0,
+                                                  _ptr(r.counts), _ptr(r.bucket), h.shape[0], ctypes.byref(m), variant,
                                                   _stream()))
     _launched()
     return r
@@ -213,14 +213,14 @@ def moe_route(h, w, b, spec: MoeSpec, counts=None) -> Routing:
 
 def moe_experts(h, gate_up, down, routing: Routing, spec: MoeSpec, variant: int = VARIANT_AUTO, status=None):
     """The chosen experts' weighted outputs [rows, top, pad8(width)] (their sum over `top` is the layer's output;
-    residual_norm takes it with parts = top).  gate_up [experts, 2, pad8(ff), pad8(width)] (gate, then up),
-    down [experts, pad8(width), pad8(ff)]."""
+    residual_norm takes it with parts = top).  gate_up [experts, pad8(ff), 2, pad8(width)] (the gate and
+    the up row of each inner column), down [experts, pad8(width), pad8(ff)]."""
     _cuda(h, gate_up, down, status)
     rows, ws = h.shape
     fs = pad8(spec.ff)
-    if tuple(gate_up.shape) != (spec.experts, 2, fs, ws) or tuple(down.shape) != (spec.experts, ws, fs) or \
+    if tuple(gate_up.shape) != (spec.experts, fs, 2, ws) or tuple(down.shape) != (spec.experts, ws, fs) or \
             gate_up.dtype != h.dtype or down.dtype != h.dtype:
-        raise ValueError("moe_experts: gate_up [experts, 2, ff stride, row stride], down [experts, row stride, ff stride]")
+        raise ValueError("moe_experts: gate_up [experts, ff stride, 2, row stride], down [experts, row stride, ff stride]")
     m = spec.c(_dtype_code(h))
     act = torch.empty(rows * spec.top, fs, dtype=h.dtype, device=h.device)
     y = torch.empty(rows, spec.top, ws, dtype=h.dtype, device=h.device)

@@ -103,7 +103,7 @@ def test_model_weights_are_padded_with_zeros_and_shapes_are_checked():
     assert q[:, 12:].abs().max() == 0 and q[:, :, 30:].abs().max() == 0
     wo = L["wo"].view(32, 2, 24)
     assert torch.equal(wo[:30, :, :20].reshape(30, 40), W["l0.mix.o"].float()) and wo[30:].abs().max() == 0
-    assert torch.equal(L["gate_up"][1, 1, :18, :30], W["l0.mlp.e1.up"].float())
+    assert torch.equal(L["gate_up"][1, :18, 1, :30], W["l0.mlp.e1.up"].float())
     assert torch.equal(L["down"][2, :30, :18], W["l0.mlp.e2.down"].float())
     lam = plain.difference_weight(*(W["l0.mix." + n].double() for n in ("lq1", "lk1", "lq2", "lk2")), 0.3)
     assert L["spec"].lam == pytest.approx(float(lam)) and L["spec"].out_scale == pytest.approx(0.7)

@@ -257,7 +257,7 @@ def _moe_case(rows, experts, top, width, ff, dtype, seed=0, skew=0.0):
     c["dev"] = lambda d: dict(
         h=p(c["h"], (0, ws - width)).to(dtype).to(d).contiguous(),
         router=p(c["router"], (0, ws - width)).to(dtype).to(d).contiguous(), b=c["b"].to(d),
-        gate_up=p(torch.stack((c["gate"], c["up"]), 1), (0, ws - width, 0, fs - ff)).to(dtype).to(d).contiguous(),
+        gate_up=p(torch.stack((c["gate"], c["up"]), 2), (0, ws - width, 0, 0, 0, fs - ff)).to(dtype).to(d).contiguous(),
         down=p(c["down"], (0, fs - ff, 0, ws - width)).to(dtype).to(d).contiguous())
     return c
 
@@ -266,13 +266,13 @@ MOE = [(1, 4, 2, 32, 24), (3, 5, 5, 72, 56), (40, 12, 3, 100, 96), (300, 7, 1, 2
        (200, 1, 1, 48, 300), (130, 3, 2, 520, 200), (77, 130, 4, 64, 32)]
 
 
-@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("dtype, variant", [(torch.float32, SIMT), (torch.bfloat16, SIMT), (torch.bfloat16, MMA)])
 @pytest.mark.parametrize("rows, experts, top, width, ff", MOE)
-def test_router(cuda_device, dtype, rows, experts, top, width, ff):
+def test_router(cuda_device, dtype, variant, rows, experts, top, width, ff):
     from kinetics_b200 import layer_ops as lo
     c = _moe_case(rows, experts, top, width, ff, dtype)
     d = c["dev"](cuda_device)
-    r = lo.moe_route(d["h"], d["router"], d["b"], lo.MoeSpec(experts, top, width, ff))
+    r = lo.moe_route(d["h"], d["router"], d["b"], lo.MoeSpec(experts, top, width, ff), variant=variant)
     z = c["h"].double() @ c["router"].double().t() + c["b"].double()
     ids = r.ids.cpu().long()
     got = z.gather(1, ids)
