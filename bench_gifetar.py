@@ -175,7 +175,7 @@ def run(args, clock_sampler):
                 perm = torch.randperm(batch * pages, device=dev, generator=gen).to(torch.int32)
                 table = lo.PageTable(perm, i32([i * pages for i in range(batch + 1)]),
                                      i32([length - (pages - 1) * ps] * batch), ps, batch * pages)
-                kp, vp = rnd(batch * pages, ps, G * 2, DIM), rnd(batch * pages, ps, G, VDIM)
+                kp, vp = rnd(batch * pages, G * 2, ps, DIM), rnd(batch * pages, G, ps, VDIM)
                 indptr = i32([0, n]) if phase == "prefill" else None
                 splits = lo.attention_splits(spec, batch, length, torch.bfloat16)
                 keys = n * (n + 1) / 2 if phase == "prefill" else batch * length

@@ -24,8 +24,8 @@
 extern "C" {
 #endif
 
-/* Paged cache of one layer:
- *   k_pages [num_pages, page_size, kv_heads * maps, dim_stride], v_pages [num_pages, page_size, kv_heads, vdim_stride]
+/* Paged cache of one layer, head by head so that a head's tokens of a page lie together:
+ *   k_pages [num_pages, kv_heads * maps, page_size, dim_stride], v_pages [num_pages, kv_heads, page_size, vdim_stride]
  * page_size is 16, 32 or 64.  CSR page table as in ktk.h, describing the state AFTER the step's append. */
 typedef struct ktk_paged {
     const int32_t* kv_indices;

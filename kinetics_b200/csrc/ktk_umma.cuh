@@ -18,6 +18,9 @@ __device__ __forceinline__ uint64_t umma_desc(uint32_t saddr, uint32_t lbo_bytes
     d |= (uint64_t)2 << 61;
     return d;
 }
+// The same descriptor `bytes` further on (a multiple of 16): the address field is the lowest, and shared memory ends
+// before it could overflow into the next one.
+__device__ __forceinline__ uint64_t umma_desc_at(uint64_t base, uint32_t bytes) { return base + (bytes >> 4); }
 // instruction descriptor of kind::f16: fp32 accumulate, bf16 A and B, A K-major, M = 128
 __device__ __forceinline__ uint32_t umma_idesc(int n, bool b_mn_major) {
     return (1u << 4) | (1u << 7) | (1u << 10) | (b_mn_major ? (1u << 16) : 0u) | ((uint32_t)(n >> 3) << 17) |
@@ -102,6 +105,16 @@ __device__ __forceinline__ void tmem_st32_u32(uint32_t taddr, const uint32_t (&v
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
+// One lane of a converged warp.  The issuing warps run their loops with all lanes and pick the lane only around the
+// instructions themselves: descriptors and barrier addresses can then stay in uniform registers, which is what the
+// tcgen05 instructions take; from a branch on the lane number every operand has to be moved there first.
+__device__ __forceinline__ bool elect_one() {
+    uint32_t on;
+    asm volatile(
+        "{\n\t.reg .pred p;\n\telect.sync _|p, 0xffffffff;\n\tselp.u32 %0, 1, 0, p;\n\t}" : "=r"(on)::"memory");
+    return on != 0;
+}
+
 // Bounded wait without a suspend-time hint: the barriers of this kernel complete within microseconds, and the
 // waiter should see that at once.  Gives up like mbar_wait (and raises *abort) after about a second of polling.
 __device__ __forceinline__ bool mbar_wait_fast(uint64_t* bar, uint32_t parity, volatile int* abort) {
@@ -129,6 +142,47 @@ __device__ __forceinline__ float ex2(float x) {
 // byte offset of the 16-byte chunk `chunk` (0..7) of row `row` in a [rows][128 B] tile under the 128-byte swizzle
 __device__ __forceinline__ uint32_t swz(int row, int chunk) {
     return (uint32_t)(row * 128 + ((chunk ^ (row & 7)) << 4));
+}
+
+// ---- two CTAs of a cluster on one tile (cta_group::2): M = 256, rows 0..127 in the first CTA's tensor memory and shared
+// memory, the rest in the second's; each stages half of B's rows; the first CTA issues ----
+__device__ __forceinline__ void umma_f16_pair(uint32_t d_tmem, uint64_t a, uint64_t b, uint32_t idesc, uint32_t accumulate) {
+    asm volatile(
+        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
+        "tcgen05.mma.cta_group::2.kind::f16 [%0], %1, %2, %3, p;\n\t}"
+        ::"r"(d_tmem), "l"(a), "l"(b), "r"(idesc), "r"(accumulate) : "memory");
+}
+__device__ __forceinline__ uint32_t umma_idesc_pair(int n) {
+    return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(n >> 3) << 17) | ((uint32_t)(2 * kUmRows >> 4) << 24);
+}
+// arrives on the barrier of this name in both CTAs
+__device__ __forceinline__ void umma_commit_pair(uint64_t* bar) {
+    const uint16_t both = 3;
+    asm volatile(
+        "tcgen05.commit.cta_group::2.mbarrier::arrive::one.shared::cluster.multicast::cluster.b64 [%0], %1;"
+        ::"r"(smem_u32(bar)), "h"(both) : "memory");
+}
+__device__ __forceinline__ void tmem_alloc_pair(uint32_t* base_smem, uint32_t cols) {
+    asm volatile("tcgen05.alloc.cta_group::2.sync.aligned.shared::cta.b32 [%0], %1;" ::"r"(smem_u32(base_smem)), "r"(cols)
+                 : "memory");
+    asm volatile("tcgen05.relinquish_alloc_permit.cta_group::2.sync.aligned;" ::: "memory");
+}
+__device__ __forceinline__ void tmem_free_pair(uint32_t base, uint32_t cols) {
+    asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, %1;" ::"r"(base), "r"(cols) : "memory");
+}
+__device__ __forceinline__ uint32_t cluster_rank() {
+    uint32_t r;
+    asm("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
+    return r;
+}
+__device__ __forceinline__ void cluster_sync() {
+    asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+}
+// arrive on the barrier of this name in CTA `cta` of the cluster
+__device__ __forceinline__ void mbar_arrive_at(uint64_t* bar, uint32_t cta) {
+    uint32_t remote;
+    asm("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(remote) : "r"(smem_u32(bar)), "r"(cta));
+    asm volatile("mbarrier.arrive.shared::cluster.b64 _, [%0];" ::"r"(remote) : "memory");
 }
 
 // Tensor memory of a CTA (one warp, all lanes): a power of two of columns >= 32, the base address into *base_smem.

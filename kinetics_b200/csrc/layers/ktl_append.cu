@@ -8,7 +8,7 @@ template <typename T>
 __global__ void __launch_bounds__(128)
 kv_append_kernel(const T* __restrict__ proj, int64_t row_stride, int64_t k_col, int64_t v_col,
                  const int32_t* __restrict__ new_indptr, T* __restrict__ k_pages, T* __restrict__ v_pages,
-                 const ktk_paged t, int k_row, int v_row, int32_t* status) {
+                 const ktk_paged t, int k_heads, int v_heads, int dim, int vdim, int32_t* status) {
     const int64_t r = blockIdx.x;
     const int b = new_indptr ? sequence_of_row(new_indptr, t.batch, r) : (int)r;
     const Span s = span_of(t, b);
@@ -22,22 +22,28 @@ kv_append_kernel(const T* __restrict__ proj, int64_t row_stride, int64_t k_col, 
         if (threadIdx.x == 0) report(status, KTK_STATUS_BAD_PAGE);
         return;
     }
-    const int64_t slot = page * t.page_size + pos % t.page_size;
+    const int slot = pos % t.page_size;
     constexpr int kPer = 16 / sizeof(T);
-    const uint4* ks = reinterpret_cast<const uint4*>(proj + r * row_stride + k_col);
-    const uint4* vs = reinterpret_cast<const uint4*>(proj + r * row_stride + v_col);
-    uint4* kd = reinterpret_cast<uint4*>(k_pages + slot * k_row);
-    uint4* vd = reinterpret_cast<uint4*>(v_pages + slot * v_row);
-    for (int i = threadIdx.x; i < k_row / kPer; i += blockDim.x) kd[i] = ks[i];
-    for (int i = threadIdx.x; i < v_row / kPer; i += blockDim.x) vd[i] = vs[i];
+    // 16-byte pieces of the row, head by head: head g of the page starts at (page * heads + g) * page_size tokens
+    auto copy = [&](const T* src, T* dst, int heads, int size) {
+        const int per = size / kPer;
+        for (int i = threadIdx.x; i < heads * per; i += blockDim.x) {
+            const int g = i / per, c = i - g * per;
+            reinterpret_cast<uint4*>(dst + (((int64_t)page * heads + g) * t.page_size + slot) * size)[c] =
+                reinterpret_cast<const uint4*>(src)[i];
+        }
+    };
+    copy(proj + r * row_stride + k_col, k_pages, k_heads, dim);
+    copy(proj + r * row_stride + v_col, v_pages, v_heads, vdim);
 }
 
 template <typename T>
 static int append_launch(const void* proj, int64_t row_stride, int64_t k_col, int64_t v_col, const int32_t* ni,
-                         int64_t rows, void* k, void* v, const ktk_paged& t, int k_row, int v_row, int32_t* status,
+                         int64_t rows, void* k, void* v, const ktk_paged& t, const ktk_attn& a, int32_t* status,
                          cudaStream_t st) {
     kv_append_kernel<T><<<(unsigned)rows, 128, 0, st>>>((const T*)proj, row_stride, k_col, v_col, ni, (T*)k, (T*)v, t,
-                                                         k_row, v_row, status);
+                                                         a.kv_heads * a.maps, a.kv_heads, a.dim_stride, a.vdim_stride,
+                                                         status);
     KTK_CUDA_TRY(cudaGetLastError(), "ktk_kv_append");
     return KTK_OK;
 }
@@ -67,10 +73,10 @@ extern "C" int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col
     }
     cudaStream_t st = (cudaStream_t)stream;
     return shape->dtype == KTK_F32
-               ? append_launch<float>(proj, row_stride, k_col, v_col, new_indptr, rows, k_pages, v_pages, *table, k_row,
-                                      v_row, status, st)
+               ? append_launch<float>(proj, row_stride, k_col, v_col, new_indptr, rows, k_pages, v_pages, *table, *shape,
+                                      status, st)
                : append_launch<__nv_bfloat16>(proj, row_stride, k_col, v_col, new_indptr, rows, k_pages, v_pages,
-                                              *table, k_row, v_row, status, st);
+                                              *table, *shape, status, st);
 }
 
 extern "C" int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int64_t max_keys) {

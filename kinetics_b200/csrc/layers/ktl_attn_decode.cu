@@ -96,16 +96,18 @@ attn_decode_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
                     continue;
                 }
                 uint8_t* dst = ring + st * kStage;
-                const int z = (int)(page * p.t.page_size) + tok % p.t.page_size;
+                const int y = tok % p.t.page_size;
                 mbar_arrive_expect_tx(&full[st], kStage);
 #pragma unroll
                 for (int mp = 0; mp < 2; ++mp)
 #pragma unroll
                     for (int c = 0; c < DC; ++c)
-                        tma_load_3d(dst + (mp * DC + c) * kAdTile, &k_map, &full[st], c * 64, kvh * 2 + mp, z);
+                        tma_load_3d(dst + (mp * DC + c) * kAdTile, &k_map, &full[st], c * 64, y,
+                                    (int)(page * (2 * a.kv_heads)) + kvh * 2 + mp);
 #pragma unroll
                 for (int c = 0; c < VC; ++c)
-                    tma_load_3d(dst + (2 * DC + c) * kAdTile, &v_map, &full[st], c * 64, kvh, z);
+                    tma_load_3d(dst + (2 * DC + c) * kAdTile, &v_map, &full[st], c * 64, y,
+                                (int)(page * a.kv_heads) + kvh);
             }
             issued_total = i;
         }
@@ -388,11 +390,19 @@ static int64_t decode_units(const ktk_attn& a, int64_t batch) {
 int32_t attn_decode_splits(const ktk_attn& a, int batch, int64_t max_keys) {
     const int64_t units = decode_units(a, batch), resident = (int64_t)sm_count() * 3;
     if (units <= 0) return 1;
-    int64_t s = (4 * resident + units - 1) / units;      // about four rounds of CTAs
-    const int64_t most = (max_keys + kAdMinKeys - 1) / kAdMinKeys;
-    if (s > most) s = most;
-    if (s > kAdMaxSplits) s = kAdMaxSplits;
-    return (int32_t)(s < 1 ? 1 : s);
+    int64_t most = (max_keys + kAdMinKeys - 1) / kAdMinKeys;
+    if (most > kAdMaxSplits) most = kAdMaxSplits;
+    // two to eight rounds of CTAs; among those the count that leaves the last round fullest
+    int64_t lo = (2 * resident + units - 1) / units, hi = (8 * resident + units - 1) / units, best = 1;
+    if (lo > most) lo = most;
+    if (hi > most) hi = most;
+    double best_fill = 0.0;
+    for (int64_t s = lo < 1 ? 1 : lo; s <= hi; ++s) {
+        const int64_t ctas = units * s, rounds = (ctas + resident - 1) / resident;
+        const double fill = (double)ctas / (double)(rounds * resident);
+        if (fill > best_fill + 0.01) { best_fill = fill; best = s; }
+    }
+    return (int32_t)best;
 }
 
 size_t attn_decode_workspace(const ktk_attn& a, int64_t rows, int splits) {
@@ -401,12 +411,13 @@ size_t attn_decode_workspace(const ktk_attn& a, int64_t rows, int splits) {
 
 int make_cache_maps(const AttnParams& p, CUtensorMap* k_map, CUtensorMap* v_map, uint32_t box_rows, const char* who) {
     const ktk_attn& a = p.a;
-    const uint64_t slots = (uint64_t)p.t.num_pages * p.t.page_size;
-    const uint64_t kr = (uint64_t)a.kv_heads * a.maps, vr = a.kv_heads;
-    const uint64_t kd[3] = {(uint64_t)a.dim_stride, kr, slots}, vd[3] = {(uint64_t)a.vdim_stride, vr, slots};
-    const uint64_t ks[2] = {(uint64_t)a.dim_stride * 2, kr * a.dim_stride * 2};
-    const uint64_t vs[2] = {(uint64_t)a.vdim_stride * 2, vr * a.vdim_stride * 2};
-    const uint32_t box[3] = {64, 1, box_rows};
+    const uint64_t ps = p.t.page_size, kr = (uint64_t)a.kv_heads * a.maps, vr = a.kv_heads;
+    // innermost first: columns, tokens of a page, (page, head)
+    const uint64_t kd[3] = {(uint64_t)a.dim_stride, ps, (uint64_t)p.t.num_pages * kr};
+    const uint64_t vd[3] = {(uint64_t)a.vdim_stride, ps, (uint64_t)p.t.num_pages * vr};
+    const uint64_t ks[2] = {(uint64_t)a.dim_stride * 2, ps * a.dim_stride * 2};
+    const uint64_t vs[2] = {(uint64_t)a.vdim_stride * 2, ps * a.vdim_stride * 2};
+    const uint32_t box[3] = {64, box_rows, 1};
     const int rc = make_tensor_map_3d(k_map, p.k, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, kd, ks, box,
                                       CU_TENSOR_MAP_SWIZZLE_128B, who);
     if (rc != KTK_OK) return rc;

@@ -30,7 +30,7 @@ template <typename T, int MAPS>
 __global__ void __launch_bounds__(kSaThreads) attn_simt_kernel(const AttnParams p) {
     extern __shared__ float sa_q[];                       // [MAPS][dim_stride]
     __shared__ float prob[MAPS][kSaThreads];
-    __shared__ int64_t key_slot[kSaThreads];
+    __shared__ int64_t key_slot[kSaThreads];              // page * page_size + slot
     __shared__ float red[4];
     const ktk_attn& a = p.a;
     const int64_t r = blockIdx.x;
@@ -67,7 +67,7 @@ __global__ void __launch_bounds__(kSaThreads) attn_simt_kernel(const AttnParams 
         for (int mp = 0; mp < MAPS; ++mp) {
             float sc = -INFINITY;
             if (slot >= 0) {
-                const T* krow = (const T*)p.k + ((slot * a.kv_heads + kvh) * MAPS + mp) * a.dim_stride;
+                const T* krow = (const T*)p.k + row_in_pages(slot, p.t.page_size, a.kv_heads * MAPS, kvh * MAPS + mp) * a.dim_stride;
                 const float* qm = sa_q + mp * a.dim_stride;
                 float d = 0.0f;
                 for (int i = 0; i < a.dim_stride; i += 8) {
@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(kSaThreads) attn_simt_kernel(const AttnParams 
         for (int i = 0; i < n; ++i) {
             const int64_t sl = key_slot[i];
             if (sl < 0) continue;
-            const T* vrow = (const T*)p.v + (sl * a.kv_heads + kvh) * a.vdim_stride;
+            const T* vrow = (const T*)p.v + row_in_pages(sl, p.t.page_size, a.kv_heads, kvh) * a.vdim_stride;
 #pragma unroll
             for (int c = 0; c < kSaCols; ++c) {
                 const int col = tid + c * kSaThreads;

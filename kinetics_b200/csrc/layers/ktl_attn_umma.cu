@@ -103,45 +103,54 @@ attn_umma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map, 
     const uint32_t tmem = tmem_base_s;
 
     if (issuer) {
-        if (lane == 0) {
-            const int ksteps = (a.dim_stride + 15) / 16;
-            const uint32_t idesc_s = umma_idesc(kAuKeys, false);
-            const uint32_t idesc_o = umma_idesc((a.vdim_stride + 15) / 16 * 16, true);
-            auto issue_s = [&](int blk) {
-                const int buf = blk & 1;
-                if (!mbar_wait_fast(&bar_k[buf], (blk >> 1) & 1, &abort_flag)) return false;
-                tc_fence_after();
+        const int ksteps = (a.dim_stride + 15) / 16;
+        const uint32_t idesc_s = umma_idesc(kAuKeys, false);
+        const uint32_t idesc_o = umma_idesc((a.vdim_stride + 15) / 16 * 16, true);
+        const uint64_t q_desc = umma_desc(smem_u32(sQ), 0, 1024), k_desc = umma_desc(smem_u32(sK), 0, 1024);
+        const uint64_t v_desc = umma_desc(smem_u32(sV), kAuVLbo, kAuVSbo);
+        auto wait = [&](uint64_t* bar, int round) {
+            return __all_sync(0xffffffffu, mbar_wait_fast(bar, round & 1, &abort_flag)) != 0;
+        };
+        auto issue_s = [&](int blk) {
+            const int buf = blk & 1;
+            if (!wait(&bar_k[buf], blk >> 1)) return false;
+            tc_fence_after();
+            if (elect_one()) {
 #pragma unroll
                 for (int m = 0; m < 2; ++m) {
-                    const uint32_t qa = smem_u32(sQ + m * DC * kAuQTile), ka = smem_u32(sK + buf * kKBuf + m * DC * kAuKTile);
+                    const uint64_t qa = umma_desc_at(q_desc, m * DC * kAuQTile);
+                    const uint64_t ka = umma_desc_at(k_desc, buf * kKBuf + m * DC * kAuKTile);
 #pragma unroll
                     for (int k = 0; k < DC * 4; ++k)
                         if (k < ksteps)
-                            umma_f16(tmem + m * 128 + buf * kAuKeys,
-                                     umma_desc(qa + (k >> 2) * kAuQTile + (k & 3) * 32, 0, 1024),
-                                     umma_desc(ka + (k >> 2) * kAuKTile + (k & 3) * 32, 0, 1024), idesc_s, k > 0 ? 1u : 0u);
+                            umma_f16(tmem + m * 128 + buf * kAuKeys, umma_desc_at(qa, (k >> 2) * kAuQTile + (k & 3) * 32),
+                                     umma_desc_at(ka, (k >> 2) * kAuKTile + (k & 3) * 32), idesc_s, k > 0 ? 1u : 0u);
                     umma_commit(&bar_s[m][buf]);
                 }
                 umma_commit(&bar_kfree[buf]);
-                return true;
-            };
-            bool ok = issue_s(0);
-            for (int j = 0; j < n_blocks && ok; ++j) {
-                const int buf = j & 1;
-                if (j + 1 < n_blocks) ok = issue_s(j + 1);
-                ok = ok && mbar_wait_fast(&bar_v[buf], (j >> 1) & 1, &abort_flag);
-                const uint32_t va = smem_u32(sV + buf * kVBuf);
+            }
+            __syncwarp();
+            return true;
+        };
+        bool ok = issue_s(0);
+        for (int j = 0; j < n_blocks && ok; ++j) {
+            const int buf = j & 1;
+            if (j + 1 < n_blocks) ok = issue_s(j + 1);
+            ok = ok && wait(&bar_v[buf], j >> 1);
+            const uint64_t va = umma_desc_at(v_desc, buf * kVBuf);
 #pragma unroll
-                for (int m = 0; m < 2; ++m) {
-                    ok = ok && mbar_wait_fast(&bar_p[m][buf], (j >> 1) & 1, &abort_flag);
-                    if (!ok) break;
-                    tc_fence_after();
+            for (int m = 0; m < 2; ++m) {
+                ok = ok && wait(&bar_p[m][buf], j >> 1);
+                if (!ok) break;
+                tc_fence_after();
+                if (elect_one()) {
 #pragma unroll
                     for (int k = 0; k < kAuKeys / 16; ++k)
                         umma_f16_ts(tmem + kAuColO + m * 128, tmem + m * 128 + buf * kAuKeys + k * 8,
-                                    umma_desc(va + k * (16 * 128), kAuVLbo, kAuVSbo), idesc_o, (j > 0 || k > 0) ? 1u : 0u);
+                                    umma_desc_at(va, k * (16 * 128)), idesc_o, (j > 0 || k > 0) ? 1u : 0u);
+                    if (m == 1) umma_commit(&bar_vfree[buf]);
                 }
-                if (ok) umma_commit(&bar_vfree[buf]);
+                __syncwarp();
             }
         }
     } else if (loader) {
@@ -152,7 +161,7 @@ attn_umma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map, 
             auto load = [&](int blk, int which) {
                 const int buf = blk & 1;
                 uint64_t* bar = which ? &bar_v[buf] : &bar_k[buf];
-                int64_t z[kAuKeys / 16];
+                int64_t z[kAuKeys / 16];                              // pages
                 uint32_t bytes = 0;
 #pragma unroll
                 for (int i = 0; i < kAuKeys / 16; ++i) {
@@ -161,7 +170,7 @@ attn_umma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map, 
                     if (i < pages && tok < seen) {
                         const int64_t pg = p.t.kv_indices[s.start + tok / ps];
                         if (pg < 0 || pg >= p.t.num_pages) report(p.status, KTK_STATUS_BAD_PAGE);
-                        else { z[i] = pg * ps; bytes += (uint32_t)((which ? VC : 2 * DC) * rows * 128); }
+                        else { z[i] = pg; bytes += (uint32_t)((which ? VC : 2 * DC) * rows * 128); }
                     }
                 }
                 if (bytes) mbar_arrive_expect_tx(bar, bytes);
@@ -172,12 +181,13 @@ attn_umma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map, 
                     if (which) {
 #pragma unroll
                         for (int c = 0; c < VC; ++c)
-                            tma_load_3d(sV + buf * kVBuf + c * kAuKTile + i * rows * 128, &v_map, bar, c * 64, kvh, (int)z[i]);
+                            tma_load_3d(sV + buf * kVBuf + c * kAuKTile + i * rows * 128, &v_map, bar, c * 64, 0,
+                                        (int)(z[i] * a.kv_heads) + kvh);
                     } else {
 #pragma unroll
                         for (int mc = 0; mc < 2 * DC; ++mc)
-                            tma_load_3d(sK + buf * kKBuf + mc * kAuKTile + i * rows * 128, &k_map, bar, (mc % DC) * 64,
-                                        kvh * 2 + mc / DC, (int)z[i]);
+                            tma_load_3d(sK + buf * kKBuf + mc * kAuKTile + i * rows * 128, &k_map, bar, (mc % DC) * 64, 0,
+                                        (int)(z[i] * (2 * a.kv_heads)) + kvh * 2 + mc / DC);
                     }
                 }
             };
@@ -228,7 +238,7 @@ attn_umma_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map, 
                     for (int c = 0; c < 32; ++c) { lo[c] = exact(lo[c]); hi[c] = exact(hi[c]); }
                 } else {
 #pragma unroll
-                    for (int c = 0; c < 32; ++c) { lo[c] = poly(lo[c]); hi[c] = poly(hi[c]); }
+                    for (int c = 0; c < 32; c += 2) { poly.two(lo[c], lo[c + 1]); poly.two(hi[c], hi[c + 1]); }
                 }
             } else {
 #pragma unroll

@@ -32,6 +32,12 @@ __device__ __forceinline__ int sequence_of_row(const int32_t* indptr, int batch,
     return lo;
 }
 
+// row of head `head` (of `heads`) at token slot `slot` = page * page_size + place, in pages stored head by head
+__device__ __forceinline__ int64_t row_in_pages(int64_t slot, int page_size, int heads, int head) {
+    const int64_t page = slot / page_size;
+    return (page * heads + head) * page_size + (slot - page * page_size);
+}
+
 // factor of the query at position pos (coef 0: none)
 __device__ __forceinline__ float query_temperature(float coef, float every, int pos) {
     if (coef == 0.0f) return 1.0f;
@@ -53,7 +59,8 @@ inline int check_attn(const ktk_attn* a, const ktk_paged* t, const char* who) {
         set_error("%s: page_size %d (16, 32 and 64 are built)", who, t->page_size);
         return KTK_ERR_UNSUPPORTED;
     }
-    if (t->batch < 0 || t->num_pages < 0 || t->num_pages > 2147483647LL / t->page_size) {
+    if (t->batch < 0 || t->num_pages < 0 || t->num_pages > 2147483647LL / t->page_size ||
+        t->num_pages > 2147483647LL / ((int64_t)a->kv_heads * a->maps)) {
         set_error("%s: batch=%d num_pages=%lld", who, t->batch, (long long)t->num_pages);
         return KTK_ERR_ARG;
     }

@@ -27,6 +27,26 @@ struct CapCoef {
 
 // The same on the FMA pipe for |s f / C| <= kPolyRange: tanh(x) = x P(x^2), P of degree 4 fitted for the smallest
 // largest relative error on that range (Remez exchange): 1.0e-6.  Coefficients are scaled per row.
+// Two fp32 operations per instruction.
+__device__ __forceinline__ uint64_t pack2(float a, float b) {
+    uint64_t r;
+    asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+    return r;
+}
+__device__ __forceinline__ void unpack2(uint64_t v, float& a, float& b) {
+    asm("mov.b64 {%0, %1}, %2;" : "=f"(a), "=f"(b) : "l"(v));
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+    uint64_t r;
+    asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+    return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+    uint64_t r;
+    asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+    return r;
+}
+
 constexpr float kPolyRange = 0.8f;
 struct CapPoly {
     float c0, c1, c2, c3, c4, limit;
@@ -43,6 +63,14 @@ struct CapPoly {
     __device__ __forceinline__ float operator()(float s) const {
         const float u = s * s;
         return s * fmaf(fmaf(fmaf(fmaf(c4, u, c3), u, c2), u, c1), u, c0);
+    }
+    __device__ __forceinline__ void two(float& a, float& b) const {
+        const uint64_t s = pack2(a, b), u = mul2(s, s);
+        uint64_t t = fma2(pack2(c4, c4), u, pack2(c3, c3));
+        t = fma2(t, u, pack2(c2, c2));
+        t = fma2(t, u, pack2(c1, c1));
+        t = fma2(t, u, pack2(c0, c0));
+        unpack2(mul2(s, t), a, b);
     }
 };
 

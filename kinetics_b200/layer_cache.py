@@ -1,8 +1,8 @@
 """KV manager for models whose layers each have their own head sizes.
 
 Pages come from the shared ``PagePool`` (``PooledTable`` keeps the slots, lengths and page tables); the cache of a
-layer is two tensors, ``k_pages [pages, page_size, kv_heads * maps, dim]`` and ``v_pages [pages, page_size, kv_heads,
-vdim]``, sized by the layer's ``AttentionSpec``.  A layer hands over its fused projection rows (queries, keys and
+layer is two tensors, ``k_pages [pages, kv_heads * maps, page_size, dim]`` and ``v_pages [pages, kv_heads, page_size,
+vdim]`` (a head's tokens of a page lie together: what one CTA reads is contiguous), sized by the layer's ``AttentionSpec``.  A layer hands over its fused projection rows (queries, keys and
 values side by side): keys and values go from there into the pages, the attention kernel reads the queries in place.
 """
 from __future__ import annotations
@@ -34,7 +34,7 @@ class LayeredKVManager(PooledTable):
         for s in self.specs:
             shape = (s.kv_heads, s.maps, s.dim_stride, s.vdim_stride)
             if not alias_layers or shape not in shared:
-                zeros = lambda *d: torch.zeros(total, page_size, *d, device=self.device, dtype=dtype)
+                zeros = lambda heads, cols: torch.zeros(total, heads, page_size, cols, device=self.device, dtype=dtype)
                 shared[shape] = (zeros(s.kv_heads * s.maps, s.dim_stride), zeros(s.kv_heads, s.vdim_stride))
             self.k_pages.append(shared[shape][0])
             self.v_pages.append(shared[shape][1])

@@ -132,8 +132,8 @@ def residual_norm(x, h, cols: int, eps: float, pre=None, y=None, parts: int = 1,
 
 
 def _cache_check(spec: AttentionSpec, table: PageTable, k_pages, v_pages):
-    if tuple(k_pages.shape) != (table.num_pages, table.page_size, spec.kv_heads * spec.maps, spec.dim_stride) or \
-            tuple(v_pages.shape) != (table.num_pages, table.page_size, spec.kv_heads, spec.vdim_stride):
+    if tuple(k_pages.shape) != (table.num_pages, spec.kv_heads * spec.maps, table.page_size, spec.dim_stride) or \
+            tuple(v_pages.shape) != (table.num_pages, spec.kv_heads, table.page_size, spec.vdim_stride):
         raise ValueError(f"cache shapes {tuple(k_pages.shape)}, {tuple(v_pages.shape)} do not fit {spec}")
 
 

@@ -103,8 +103,8 @@ class PagedCase:
             if n:
                 K[slots] = torch.nn.functional.pad(k.reshape(n, Gm, d), (0, pad8(d) - d))
                 V[slots] = torch.nn.functional.pad(v, (0, pad8(dv) - dv))
-        self.k = K.view(total, ps, Gm, pad8(d)).to(dtype).to(device)
-        self.v = V.view(total, ps, G, pad8(dv)).to(dtype).to(device)
+        pages_of = lambda t, heads, cols: t.view(total, ps, heads, cols).transpose(1, 2).contiguous().to(dtype).to(device)
+        self.k, self.v = pages_of(K, Gm, pad8(d)), pages_of(V, G, pad8(dv))
         i32 = lambda x: torch.tensor(x, dtype=torch.int32, device=device)
         self.table = PageTable(i32(idx or [0]), i32(indptr), i32(last), ps, total)
 

@@ -154,7 +154,7 @@ def test_layered_manager_bookkeeping_on_the_host():
     from kinetics_b200.layer_ops import AttentionSpec
     specs = [AttentionSpec(4, 2, 24, 40, 0.1, maps=2), AttentionSpec(2, 1, 8, 8, 0.1, maps=2)]
     kv = LayeredKVManager(specs, 3, 200, "cpu", torch.float32, num_pages=8, page_size=16)
-    assert tuple(kv.k_pages[0].shape) == (8, 16, 4, 24) and tuple(kv.v_pages[1].shape) == (8, 16, 1, 8)
+    assert tuple(kv.k_pages[0].shape) == (8, 4, 16, 24) and tuple(kv.v_pages[1].shape) == (8, 1, 16, 8)
     assert kv.can_admit(128) and not kv.can_admit(129)
     kv.admit(0, 0, 40)
     kv.admit(1, 0, 0)

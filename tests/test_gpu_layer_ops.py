@@ -69,7 +69,8 @@ def test_append_writes_rows_into_their_pages(cuda_device, dtype, page):
     status = ops.new_status(cuda_device)
     lo.kv_append(proj, spec.q_cols, spec.q_cols + spec.k_cols, case.k, case.v, case.table, spec, indptr, status=status)
     idx, ptr, _ = (t.cpu() for t in case.table.tensors)
-    want_k, want_v = before_k.cpu().view(-1, spec.k_cols), before_v.cpu().view(-1, spec.v_cols)
+    tokens = lambda t: t.cpu().transpose(1, 2).reshape(t.shape[0] * page, -1)       # token slot by token slot
+    want_k, want_v = tokens(before_k), tokens(before_v)
     r = 0
     for b, n in enumerate(new):
         for t in range(lens[b] - n, lens[b]):
@@ -78,14 +79,14 @@ def test_append_writes_rows_into_their_pages(cuda_device, dtype, page):
             want_v[slot] = proj[r, spec.q_cols + spec.k_cols:].cpu()
             r += 1
     same = lambda a, b: torch.equal(torch.nan_to_num(a.float(), nan=7.0), torch.nan_to_num(b.float(), nan=7.0))
-    assert same(case.k.cpu().view(-1, spec.k_cols), want_k) and same(case.v.cpu().view(-1, spec.v_cols), want_v)
+    assert same(tokens(case.k), want_k) and same(tokens(case.v), want_v)
     # one row per sequence: the newest token of each
     one = torch.randn(4, proj.shape[1]).to(dtype).to(cuda_device)
     lo.kv_append(one, spec.q_cols, spec.q_cols + spec.k_cols, case.k, case.v, case.table, spec, status=status)
     for b in range(4):
         t = lens[b] - 1
         slot = int(idx[ptr[b] + t // page]) * page + t % page
-        assert torch.equal(case.k.view(-1, spec.k_cols)[slot], one[b, spec.q_cols:spec.q_cols + spec.k_cols])
+        assert torch.equal(tokens(case.k)[slot], one[b, spec.q_cols:spec.q_cols + spec.k_cols].cpu())
     assert int(status.item()) == 0
 
 
@@ -263,7 +264,8 @@ def _moe_case(rows, experts, top, width, ff, dtype, seed=0, skew=0.0):
 
 
 MOE = [(1, 4, 2, 32, 24), (3, 5, 5, 72, 56), (40, 12, 3, 100, 96), (300, 7, 1, 256, 130), (513, 64, 8, 136, 64),
-       (200, 1, 1, 48, 300), (130, 3, 2, 520, 200), (77, 130, 4, 64, 32)]
+       (200, 1, 1, 48, 300), (130, 3, 2, 520, 200), (77, 130, 4, 64, 32),
+       (700, 3, 2, 200, 176), (520, 1, 1, 72, 40), (900, 2, 2, 264, 520), (257, 1, 1, 64, 128)]
 
 
 @pytest.mark.parametrize("dtype, variant", [(torch.float32, SIMT), (torch.bfloat16, SIMT), (torch.bfloat16, MMA)])
