@@ -508,6 +508,8 @@ class Engine:
             raise ValueError(f"slot {slot} is not open")
         ids = torch.as_tensor(tokens, dtype=torch.long).reshape(1, -1).to(self.device)
         n, held = ids.shape[1], self._offsets_host[slot]
+        if n == 0:
+            return None
         if held + n > self.max_seq_len:
             raise ValueError(f"{held} + {n} tokens exceed max_seq_len {self.max_seq_len}")
         if hasattr(self.kv, "promise"):

@@ -1,6 +1,5 @@
 """The plain Gifetar restatement itself, the configuration and weight reader, and the command line's host side.  No
 GPU."""
-import io
 import json
 import math
 
