@@ -47,20 +47,22 @@ typedef struct ktk_attn {
     float softcap;                   /* > 0: score <- softcap * tanh(score / softcap)            */
     float temp_coef, temp_every;     /* temperature at position p: 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) */
     float lambda, eps, out_scale;    /* maps = 2 */
+    int32_t v_row_stride;            /* 0: v_pages as above.  dim_stride: a key row's first vdim columns are the value
+                                        (v_pages = k_pages), as in attention over latents                */
 } ktk_attn;
 
 /*
  * One pass over rows of the fp32 residual stream x [rows, stride]:
- *   start:   x = embed[token] (tokens and embed given; x is then only written), or x as it lies
+ *   start:   x = embed[token] * embed_scale (tokens and embed given; x is then only written), or x as it lies
  *   add:     y given: s = sum over `parts` of y[row, part, :];  x += mult * norm(s; post_w, post_b), or
  *            x += mult * s where post_w is null
- *   output:  h given: h = norm(x; pre_w, pre_b), in `dtype`
+ *   output:  h given: h = norm(x; pre_w, pre_b), or x itself where pre_w is null, in `dtype`
  * norm(v; w, b) = (v - c) / sqrt(mean((v - c)^2) + eps) * w + b over the first `cols` columns, with c the mean of v
  * (center != 0) or 0, and b null for none.  Norm weights are fp32 [stride].
  * zero (nullable): zero_n ints that the launch clears (the expert counters of the router behind it).
  */
-KTK_API int ktk_residual_norm(const int64_t* tokens, const void* embed, int64_t vocab, float* x, const void* y,
-                              int32_t parts, const float* post_w, const float* post_b, float mult, const float* pre_w,
+KTK_API int ktk_residual_norm(const int64_t* tokens, const void* embed, int64_t vocab, float embed_scale, float* x,
+                              const void* y, int32_t parts, const float* post_w, const float* post_b, float mult, const float* pre_w,
                               const float* pre_b, void* h, float eps, int32_t center, int64_t rows, int32_t cols,
                               int32_t stride, int32_t* zero, int32_t zero_n, int32_t dtype, int32_t* status,
                               void* stream);
@@ -79,13 +81,68 @@ KTK_API int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col, i
  * q [rows, q_stride]: heads * maps * dim_stride columns, head by head and map by map; o [rows, heads * vdim_stride].
  * variant: KTK_VARIANT_AUTO, _SIMT (any size, fp32 math), _MMA (bf16, one row per sequence), _UMMA (bf16 on tcgen05).
  * splits: parts that a sequence's keys are cut into where new_indptr is null (0: policy).
+ * sink fp32 [heads] (nullable, maps = 1): exp(sink) joins each row's denominator, without key, value or scale.
+ * gate (nullable, maps = 1), in `dtype`: head h of row r is multiplied by sigmoid(gate[r * gate_stride + h]).
  */
 KTK_API int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int64_t max_keys);
 KTK_API size_t ktk_paged_attention_workspace(const ktk_attn* shape, int64_t rows, int32_t splits);
 KTK_API int ktk_paged_attention(const void* q, int64_t q_stride, const int32_t* new_indptr, int64_t rows,
                                 int32_t max_new, const void* k_pages, const void* v_pages, const ktk_paged* table,
-                                void* o, void* workspace, size_t workspace_bytes, int32_t splits, int32_t variant,
-                                const ktk_attn* shape, int32_t* status, void* stream);
+                                const float* sink, const void* gate, int64_t gate_stride, void* o, void* workspace,
+                                size_t workspace_bytes, int32_t splits, int32_t variant, const ktk_attn* shape,
+                                int32_t* status, void* stream);
+
+/*
+ * Latent attention: heads share one cached row per token, [latent (rank_stride) | rotated key (rot_stride)]; the page
+ * tensor is [num_pages, page_size, rank_stride + rot_stride].  The attention itself is ktk_paged_attention over those
+ * rows (kv_heads = 1, dim = rank_stride + rot_stride, vdim = rank, v_row_stride = dim_stride) with queries that carry
+ * the key expansion, or ktk_expanded_attention.
+ */
+typedef struct ktk_latent {
+    int32_t heads, dim, rot_dim, vdim, rank;              /* true sizes; dim: the unrotated part of a query head */
+    int32_t dim_stride, rot_stride, vdim_stride, rank_stride;
+    int32_t dtype;
+    float scale;
+    float eps;                                            /* of the latent's norm */
+    float rot_factor;                                     /* of cos and sin */
+} ktk_latent;
+
+/*
+ * One launch per layer over rows of proj [rows, row_stride]:
+ *   queries at q_col: heads of [dim_stride | rot_stride]; the rotated part (pairs 2 i, 2 i + 1 turned by position *
+ *   freqs[i], fp32 [rot_dim / 2]) goes to q_out [rows, heads, rank_stride + rot_stride], columns rank_stride.., or back
+ *   in place where q_out is null;
+ *   latents at kv_col (< 0: none): [rank_stride | rot_stride]; norm(latent) * norm_w (fp32 [rank_stride]) and the
+ *   rotated key go to the token's page row.
+ */
+KTK_API int ktk_latent_append(void* proj, int64_t row_stride, int64_t q_col, int64_t kv_col, const int32_t* new_indptr,
+                              int64_t rows, const float* norm_w, const float* freqs, void* q_out, void* pages,
+                              const ktk_paged* table, const ktk_latent* shape, int32_t* status, void* stream);
+
+/* Linear recurrence with real gates, per channel (blocks of block_stride channels, the first `block` of them real):
+ *   u = conv_b + sum_k conv_w[k] x_(t - taps + 1 + k)                     causal, zeros before the sequence
+ *   r = sigmoid(zr + rb), i = sigmoid(zi + ib)                            zr, zi: block-diagonal products of u
+ *   a = exp(-r decay);  S <- a S + sqrt(1 - a^2) i u;  out = S gelu_tanh(y)
+ * `state` fp32 [slots, width] and `ring` [slots, taps, width] (the newest inputs, that of position p at p % taps) belong
+ * to slots; a sequence that starts at position 0 reads neither.  width = blocks * block_stride.
+ */
+typedef struct ktk_lru {
+    int32_t blocks, block, block_stride, taps;
+    int32_t dtype;
+} ktk_lru;
+
+/* x: rows of proj at column x_col; u [rows, width]; conv_w fp32 [taps, width], conv_b fp32 [width].  slots int32 [batch];
+ * new_indptr as in ktk_kv_append.  Updates the ring. */
+KTK_API int ktk_lru_conv(const void* proj, int64_t row_stride, int64_t x_col, const int32_t* new_indptr, int64_t rows,
+                         int32_t max_new, const int32_t* slots, int64_t num_slots, const float* conv_w,
+                         const float* conv_b, void* ring, void* u, const ktk_paged* table, const ktk_lru* shape,
+                         int32_t* status, void* stream);
+
+/* z fp32 [blocks, rows, 2 * block_stride]: zr, then zi of a block; y: rows of proj at y_col; out [rows, width] in dtype. */
+KTK_API int ktk_lru_scan(const float* z, const void* u, const void* proj, int64_t row_stride, int64_t y_col,
+                         const int32_t* new_indptr, int64_t rows, int32_t max_new, const int32_t* slots,
+                         int64_t num_slots, const float* rb, const float* ib, const float* decay, float* state,
+                         void* out, const ktk_paged* table, const ktk_lru* shape, int32_t* status, void* stream);
 
 /* Mixture of experts over rows h [rows, width_stride]. */
 typedef struct ktk_moe {
@@ -93,12 +150,13 @@ typedef struct ktk_moe {
     int32_t width, ff;               /* true sizes */
     int32_t width_stride, ff_stride;
     int32_t dtype;
-    int32_t reserved;
+    int32_t scoring;                 /* weights: 0 softmax over the chosen logits, 1 softmax over all of them */
+    float limit, slope, shift;       /* gated activation, see ktk_gated_rows */
 } ktk_moe;
 
 /*
- * logits = W h + b in fp32 (W [experts, width_stride], b fp32); the `top` largest of each row (ties to the lower
- * expert), weights = softmax over those.  ids / weights [rows, top].  counts [experts] (cleared by the caller):
+ * logits = W h + b in fp32 (W [experts, width_stride], b fp32 or null); the `top` largest of each row (ties to the
+ * lower expert) and their weights (`scoring`).  ids / weights [rows, top].  counts [experts] (cleared by the caller):
  * rows of each expert; bucket [experts, rows]: their row * top + place, in no particular order.
  */
 KTK_API int ktk_moe_route(const void* h, const void* w, const float* b, int32_t* ids, float* weights, int32_t* counts,
@@ -106,7 +164,7 @@ KTK_API int ktk_moe_route(const void* h, const void* w, const float* b, int32_t*
 
 /*
  * Expert products.  Rows of expert e take the places [sum of counts before e, + counts[e]) of `act`.
- *   stage 0: act [rows * top, ff_stride] = silu(G h) * (U h);  w = [experts, ff_stride, 2, width_stride] (a row of G, then
+ *   stage 0: act [rows * top, ff_stride] = gated(G h, U h);  w = [experts, ff_stride, 2, width_stride] (a row of G, then
  *            the row of U of the same inner column)
  *   stage 1: y [rows, top, width_stride] = weight * (D act);   w = [experts, width_stride, ff_stride]
  * variant: KTK_VARIANT_AUTO, _SIMT (fp32 math), _UMMA (bf16 on tcgen05).
@@ -114,6 +172,17 @@ KTK_API int ktk_moe_route(const void* h, const void* w, const float* b, int32_t*
 KTK_API int ktk_moe_gemm(int32_t stage, const void* in, const void* w, void* out, const float* weights,
                          const int32_t* counts, const int32_t* bucket, int64_t rows, const ktk_moe* shape,
                          int32_t variant, int32_t* status, void* stream);
+
+/*
+ * out [rows, cols_stride] = gated(in[:, 0 .. cols_stride), in[:, cols_stride .. 2 cols_stride)):
+ *   gated(g, u) = g' sigmoid(slope g') (u' + shift),  g' = min(g, limit),  u' = clamp(u, -limit, limit)
+ * (limit = infinity, slope = 1, shift = 0: silu(g) u).
+ */
+KTK_API int ktk_gated_rows(const void* in, void* out, int64_t rows, int32_t cols_stride, float limit, float slope,
+                           float shift, int32_t dtype, void* stream);
+
+/* z [n] <- cap tanh(z scale / cap), fp32, in place (cap <= 0: z scale). */
+KTK_API int ktk_scale_cap(float* z, int64_t n, float scale, float cap, void* stream);
 
 #ifdef __cplusplus
 }

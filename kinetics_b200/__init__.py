@@ -20,8 +20,9 @@ from .engine import Engine, PagePool, PooledKVManager, PoolExhausted  # noqa: E4
 from .decoder_stack import DecoderStack  # noqa: E402
 from .layer_cache import LayeredKVManager  # noqa: E402
 from .gifetar import Gifetar, GifetarConfig  # noqa: E402
+from .munadra import Munadra, MunadraConfig  # noqa: E402
 from .registry import load_model, model_class  # noqa: E402
 
 __all__ = ["ops", "LayerConfig", "get_config", "BlockTopkDecoderLayer", "DecoderLayer", "init_weights",
            "BatchKVManager", "DecoderStack", "Engine", "Gifetar", "GifetarConfig", "LayeredKVManager", "load_model",
-           "model_class", "PagePool", "PooledKVManager", "PoolExhausted"]
+           "model_class", "Munadra", "MunadraConfig", "PagePool", "PooledKVManager", "PoolExhausted"]

@@ -46,13 +46,26 @@ class Attn(ctypes.Structure):
     """ktk_attn"""
     _fields_ = [(n, c_int32) for n in ("heads", "kv_heads", "maps", "dim", "vdim", "dim_stride", "vdim_stride",
                                        "dtype")] + \
-               [(n, c_float) for n in ("scale", "softcap", "temp_coef", "temp_every", "lam", "eps", "out_scale")]
+               [(n, c_float) for n in ("scale", "softcap", "temp_coef", "temp_every", "lam", "eps", "out_scale")] + \
+               [("v_row_stride", c_int32)]
 
 
 class Moe(ctypes.Structure):
     """ktk_moe"""
     _fields_ = [(n, c_int32) for n in ("experts", "top", "width", "ff", "width_stride", "ff_stride", "dtype",
-                                       "reserved")]
+                                       "scoring")] + [(n, c_float) for n in ("limit", "slope", "shift")]
+
+
+class Latent(ctypes.Structure):
+    """ktk_latent"""
+    _fields_ = [(n, c_int32) for n in ("heads", "dim", "rot_dim", "vdim", "rank", "dim_stride", "rot_stride",
+                                       "vdim_stride", "rank_stride", "dtype")] + \
+               [(n, c_float) for n in ("scale", "eps", "rot_factor")]
+
+
+class Lru(ctypes.Structure):
+    """ktk_lru"""
+    _fields_ = [(n, c_int32) for n in ("blocks", "block", "block_stride", "taps", "dtype")]
 
 
 class View(ctypes.Structure):
@@ -147,7 +160,7 @@ _SIGNATURES = {
 }
 
 _LAYER_SIGNATURES = {
-    "ktk_residual_norm": (c_int32, [c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_int32, c_void_p, c_void_p,
+    "ktk_residual_norm": (c_int32, [c_void_p, c_void_p, c_int64, c_float, c_void_p, c_void_p, c_int32, c_void_p, c_void_p,
                                     c_float, c_void_p, c_void_p, c_void_p, c_float, c_int32, c_int64, c_int32, c_int32,
                                     _i32p, c_int32, c_int32, _i32p, c_void_p]),
     "ktk_kv_append": (c_int32, [c_void_p, c_int64, c_int64, c_int64, _i32p, c_int64, c_void_p, c_void_p,
@@ -155,7 +168,16 @@ _LAYER_SIGNATURES = {
     "ktk_paged_attention_splits": (c_int32, [POINTER(Attn), c_int32, c_int64]),
     "ktk_paged_attention_workspace": (c_size_t, [POINTER(Attn), c_int64, c_int32]),
     "ktk_paged_attention": (c_int32, [c_void_p, c_int64, _i32p, c_int64, c_int32, c_void_p, c_void_p, POINTER(Paged),
-                                      c_void_p, c_void_p, c_size_t, c_int32, c_int32, POINTER(Attn), _i32p, c_void_p]),
+                                      c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_size_t, c_int32, c_int32, POINTER(Attn), _i32p, c_void_p]),
+    "ktk_latent_append": (c_int32, [c_void_p, c_int64, c_int64, c_int64, _i32p, c_int64, c_void_p, c_void_p, c_void_p,
+                                    c_void_p, POINTER(Paged), POINTER(Latent), _i32p, c_void_p]),
+    "ktk_lru_conv": (c_int32, [c_void_p, c_int64, c_int64, _i32p, c_int64, c_int32, _i32p, c_int64, c_void_p, c_void_p,
+                               c_void_p, c_void_p, POINTER(Paged), POINTER(Lru), _i32p, c_void_p]),
+    "ktk_lru_scan": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_int64, _i32p, c_int64, c_int32, _i32p, c_int64,
+                               c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, POINTER(Paged), POINTER(Lru), _i32p,
+                               c_void_p]),
+    "ktk_gated_rows": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_float, c_float, c_float, c_int32, c_void_p]),
+    "ktk_scale_cap": (c_int32, [c_void_p, c_int64, c_float, c_float, c_void_p]),
     "ktk_moe_route": (c_int32, [c_void_p, c_void_p, c_void_p, _i32p, c_void_p, _i32p, _i32p, c_int64, POINTER(Moe),
                                 c_int32, c_void_p]),
     "ktk_moe_gemm": (c_int32, [c_int32, c_void_p, c_void_p, c_void_p, c_void_p, _i32p, _i32p, c_int64, POINTER(Moe),

@@ -71,6 +71,7 @@ extern "C" int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col
         set_error("%s: null or misaligned pointer, or columns outside the row", who);
         return KTK_ERR_ARG;
     }
+    if (shape->v_row_stride != 0) { set_error("%s: values inside the keys are written by ktk_latent_append", who); return KTK_ERR_UNSUPPORTED; }
     cudaStream_t st = (cudaStream_t)stream;
     return shape->dtype == KTK_F32
                ? append_launch<float>(proj, row_stride, k_col, v_col, new_indptr, rows, k_pages, v_pages, *table, *shape,
@@ -89,8 +90,9 @@ extern "C" size_t ktk_paged_attention_workspace(const ktk_attn* shape, int64_t r
 
 extern "C" int ktk_paged_attention(const void* q, int64_t q_stride, const int32_t* new_indptr, int64_t rows,
                                    int32_t max_new, const void* k_pages, const void* v_pages, const ktk_paged* table,
-                                   void* o, void* workspace, size_t workspace_bytes, int32_t splits, int32_t variant,
-                                   const ktk_attn* shape, int32_t* status, void* stream) {
+                                   const float* sink, const void* gate, int64_t gate_stride, void* o, void* workspace,
+                                   size_t workspace_bytes, int32_t splits, int32_t variant, const ktk_attn* shape,
+                                   int32_t* status, void* stream) {
     const char* who = "ktk_paged_attention";
     const int rc = check_attn(shape, table, who);
     if (rc != KTK_OK) return rc;
@@ -110,8 +112,10 @@ extern "C" int ktk_paged_attention(const void* q, int64_t q_stride, const int32_
         set_error("%s: unknown variant %d", who, variant);
         return KTK_ERR_ARG;
     }
-    AttnParams p{*shape, *table, q, q_stride, new_indptr, rows, max_new, k_pages, v_pages, o, (float*)workspace, splits,
-                 status};
+    if ((sink || gate) && shape->maps != 1) { set_error("%s: sinks and gates go with one map", who); return KTK_ERR_UNSUPPORTED; }
+    if (gate && gate_stride < shape->heads) { set_error("%s: gate_stride %lld", who, (long long)gate_stride); return KTK_ERR_ARG; }
+    AttnParams p{*shape, *table, q, q_stride, new_indptr, rows, max_new, k_pages, v_pages, sink, gate, gate_stride, o,
+                 (float*)workspace, splits, status};
     const bool can_decode = !new_indptr && attn_decode_supported(*shape);
     const bool can_umma = new_indptr && attn_umma_supported(*shape);
     if ((variant == KTK_VARIANT_MMA && !can_decode) || (variant == KTK_VARIANT_UMMA && !can_umma)) {

@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(kSaThreads) attn_simt_kernel(const AttnParams 
         for (int i = 0; i < n; ++i) {
             const int64_t sl = key_slot[i];
             if (sl < 0) continue;
-            const T* vrow = (const T*)p.v + row_in_pages(sl, p.t.page_size, a.kv_heads, kvh) * a.vdim_stride;
+            const T* vrow = (const T*)p.v + row_in_pages(sl, p.t.page_size, a.kv_heads, kvh) * value_row(a);
 #pragma unroll
             for (int c = 0; c < kSaCols; ++c) {
                 const int col = tid + c * kSaThreads;
@@ -106,6 +106,13 @@ __global__ void __launch_bounds__(kSaThreads) attn_simt_kernel(const AttnParams 
         }
         __syncthreads();
     }
+    if (MAPS == 1 && p.sink != nullptr) {
+        const float sk = p.sink[head], mn = fmaxf(m[0], sk);
+        const float old = expf(m[0] - mn);
+        l[0] = l[0] * old + expf(sk - mn);
+#pragma unroll
+        for (int c = 0; c < kSaCols; ++c) acc[0][c] *= old;
+    }
     T* dst = (T*)p.o + (r * a.heads + head) * a.vdim_stride;
     float o[kSaCols], ss = 0.0f;
 #pragma unroll
@@ -115,6 +122,7 @@ __global__ void __launch_bounds__(kSaThreads) attn_simt_kernel(const AttnParams 
         if (tid + c * kSaThreads < a.vdim) ss += o[c] * o[c];
     }
     float f = 1.0f;
+    if (MAPS == 1 && p.gate != nullptr) f = sigmoid_f(to_f32(((const T*)p.gate)[r * p.gate_stride + head]));
     if (MAPS == 2) f = a.out_scale / sqrtf(cta_sum(ss, red) / (float)a.vdim + a.eps);
 #pragma unroll
     for (int c = 0; c < kSaCols; ++c) {

@@ -49,7 +49,8 @@ inline int check_attn(const ktk_attn* a, const ktk_paged* t, const char* who) {
     if (a->heads <= 0 || a->kv_heads <= 0 || a->heads % a->kv_heads != 0 || a->dim <= 0 || a->vdim <= 0 ||
         a->dim_stride < a->dim || a->vdim_stride < a->vdim || a->dim_stride % 8 != 0 || a->vdim_stride % 8 != 0 ||
         (a->maps != 1 && a->maps != 2) || (a->dtype != KTK_F32 && a->dtype != KTK_BF16) ||
-        (a->temp_coef != 0.0f && !(a->temp_every > 0.0f))) {
+        (a->temp_coef != 0.0f && !(a->temp_every > 0.0f)) ||
+        (a->v_row_stride != 0 && (a->v_row_stride != a->dim_stride || a->vdim_stride > a->dim_stride || a->maps != 1))) {
         set_error("%s: heads=%d kv_heads=%d maps=%d dim=%d (stride %d) vdim=%d (stride %d) dtype=%d temp_every=%g", who,
                   a->heads, a->kv_heads, a->maps, a->dim, a->dim_stride, a->vdim, a->vdim_stride, a->dtype,
                   (double)a->temp_every);
@@ -67,6 +68,11 @@ inline int check_attn(const ktk_attn* a, const ktk_paged* t, const char* who) {
     return KTK_OK;
 }
 
+// elements between two value rows of a head
+__host__ __device__ __forceinline__ int value_row(const ktk_attn& a) { return a.v_row_stride ? a.v_row_stride : a.vdim_stride; }
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf(-x)); }
+
 struct AttnParams {
     ktk_attn a;
     ktk_paged t;
@@ -76,11 +82,38 @@ struct AttnParams {
     int64_t rows;
     int max_new;
     const void *k, *v;
+    const float* sink;
+    const void* gate;
+    int64_t gate_stride;
     void* o;
     float* ws;
     int splits;
     int32_t* status;
 };
+
+// latent attention: its sizes, and the attention over its cached rows
+inline int check_latent(const ktk_latent* a, const char* who) {
+    if (a == nullptr || a->heads <= 0 || a->dim <= 0 || a->rot_dim < 0 || a->rot_dim % 2 != 0 || a->vdim <= 0 || a->rank <= 0 ||
+        a->dim_stride < a->dim || a->rot_stride < a->rot_dim || a->vdim_stride < a->vdim || a->rank_stride < a->rank ||
+        (a->dim_stride | a->rot_stride | a->vdim_stride | a->rank_stride) % 8 != 0 || a->rot_stride > 4096 ||
+        (a->dtype != KTK_F32 && a->dtype != KTK_BF16)) {
+        set_error("%s: bad sizes", who);
+        return KTK_ERR_ARG;
+    }
+    return KTK_OK;
+}
+inline ktk_attn latent_rows(const ktk_latent& a) {
+    ktk_attn r{};
+    r.heads = a.heads;
+    r.kv_heads = r.maps = 1;
+    r.dim = r.dim_stride = r.v_row_stride = a.rank_stride + a.rot_stride;
+    r.vdim = a.rank;
+    r.vdim_stride = a.rank_stride;
+    r.dtype = a.dtype;
+    r.scale = a.scale;
+    r.temp_every = 1.0f;
+    return r;
+}
 
 int launch_attn_simt(const AttnParams& p, cudaStream_t st);
 bool attn_decode_supported(const ktk_attn& a);
@@ -108,6 +141,15 @@ struct MoeParams {
 int launch_moe_simt(int stage, const MoeParams& p, cudaStream_t st);
 bool moe_umma_supported(const ktk_moe& m);
 int launch_moe_umma(int stage, const MoeParams& p, cudaStream_t st);
+
+// g' sigmoid(slope g') (u' + shift), g' = min(g, limit), u' = clamp(u, -limit, limit).  FAST: with the special-function
+// unit's exponential.
+template <bool FAST> __device__ __forceinline__ float gated(float g, float u, float limit, float slope, float shift) {
+    g = fminf(g, limit);
+    u = fminf(fmaxf(u, -limit), limit) + shift;
+    if (FAST) return __fdividef(g, 1.0f + __expf(-slope * g)) * u;
+    return g / (1.0f + expf(-slope * g)) * u;
+}
 
 // How the rows of all experts are cut into tiles of at most `tile` rows; one warp fills this from `counts`.
 struct ExpertPlan {

@@ -1,0 +1,317 @@
+// A linear recurrence with real gates behind a short causal convolution, per channel (see ktk_layers.h), over a
+// sequence's next tokens or one token of every sequence.  State, gates and decays are fp32.
+//
+// The convolution keeps its newest `taps` inputs in a ring by position: a step writes the place of the input that has
+// just left the window, which nobody reads.  The prompt's scan is one pass: a CTA owns 16 channels and walks the tokens
+// in tiles; a thread runs 8 tokens of a channel, a warp shuffle joins the 16 runs of a tile, and the carry stays in a
+// register.  The next tile's loads are in flight meanwhile.
+#include "ktl_common.cuh"
+
+namespace ktk {
+
+constexpr int kLcThreads = 64;
+constexpr int kLcChunk = 16;            // tokens per thread of the convolution
+constexpr int kLsChan = 16, kLsSegs = 16, kLsRun = 8;
+constexpr int kLsThreads = kLsChan * kLsSegs, kLsTile = kLsSegs * kLsRun;
+constexpr int kLdThreads = 128;
+
+// what a sequence runs now: rows [row0, row0 + n), of positions base ..; false if the table or the slot is malformed
+struct Run { int64_t row0; int n, base, slot; };
+__device__ __forceinline__ bool run_of(const ktk_paged& t, const int32_t* new_indptr, const int32_t* slots, int64_t num_slots,
+                                       int b, int32_t* status, Run& r) {
+    const Span s = span_of(t, b);
+    r.row0 = new_indptr ? new_indptr[b] : b;
+    r.n = new_indptr ? new_indptr[b + 1] - new_indptr[b] : 1;
+    r.base = s.total - r.n;
+    r.slot = slots[b];
+    const bool ok = !s.bad && r.base >= 0 && r.slot >= 0 && r.slot < num_slots;
+    if (!ok && threadIdx.x == 0) report(status, KTK_STATUS_BAD_TABLE);
+    return ok;
+}
+
+// Thread: 8 channels of `chunk` tokens.  TAPS > 0: the window stays in registers; 0: any number of taps.
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(kLcThreads)
+lru_conv_kernel(const T* __restrict__ x, int64_t row_stride, const int32_t* __restrict__ new_indptr,
+                const int32_t* __restrict__ slots, int64_t num_slots, const float* __restrict__ w, const float* __restrict__ bias,
+                T* ring, T* __restrict__ u, const ktk_paged t, int width, int taps_any, int chunk, int32_t* status) {
+    Run r;
+    if (!run_of(t, new_indptr, slots, num_slots, blockIdx.z, status, r)) return;
+    const int taps = TAPS > 0 ? TAPS : taps_any;
+    const int c = (blockIdx.x * kLcThreads + threadIdx.x) * 8;
+    const int t0 = blockIdx.y * chunk, t1 = t0 + chunk < r.n ? t0 + chunk : r.n;
+    if (c >= width || t0 >= r.n) return;
+    T* mine = ring + (int64_t)r.slot * taps * width + c;
+    auto input = [&](int i, float (&v)[8]) {              // input of token i of the run (i < 0: an earlier one)
+        if (i >= 0) Vec8<T>::load(x + (r.row0 + i) * row_stride + c, v);
+        else if (r.base + i >= 0) Vec8<T>::load(mine + (int64_t)((r.base + i) % taps) * width, v);
+        else {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] = 0.0f;
+        }
+    };
+    float b8[8];
+    load8(bias + c, b8);
+    if (TAPS > 0) {
+        float win[TAPS > 0 ? TAPS : 1][8], wt[TAPS > 0 ? TAPS : 1][8];
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) {
+            load8(w + (int64_t)k * width + c, wt[k]);
+            if (k + 1 < TAPS) input(t0 - (TAPS - 1) + k, win[k]);
+        }
+        for (int i = t0; i < t1; ++i) {
+            input(i, win[TAPS > 0 ? TAPS - 1 : 0]);
+            float o[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = b8[e];
+#pragma unroll
+            for (int k = 0; k < TAPS; ++k)
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    o[e] = fmaf(wt[k][e], win[k][e], o[e]);
+                    if (k > 0) win[k - 1][e] = win[k][e];
+                }
+            Vec8<T>::store(u + (r.row0 + i) * width + c, o);
+        }
+    } else {
+        for (int i = t0; i < t1; ++i) {
+            float o[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) o[e] = b8[e];
+            for (int k = 0; k < taps; ++k) {
+                float v[8], wk[8];
+                input(i - (taps - 1) + k, v);
+                load8(w + (int64_t)k * width + c, wk);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) o[e] = fmaf(wk[e], v[e], o[e]);
+            }
+            Vec8<T>::store(u + (r.row0 + i) * width + c, o);
+        }
+    }
+    // the first chunk's thread is the only one that reads this ring (a chunk has at least `taps` tokens): it also writes
+    if (t0 == 0)
+        for (int i = r.n > taps ? r.n - taps : 0; i < r.n; ++i) {
+            float v[8];
+            Vec8<T>::load(x + (r.row0 + i) * row_stride + c, v);
+            Vec8<T>::store(mine + (int64_t)((r.base + i) % taps) * width, v);
+        }
+}
+
+// ---- gates and the recurrence ----
+template <bool FAST> __device__ __forceinline__ float exp_of(float x) { return FAST ? __expf(x) : expf(x); }
+template <bool FAST> __device__ __forceinline__ float sigmoid_of(float x) {
+    return FAST ? __fdividef(1.0f, 1.0f + __expf(-x)) : 1.0f / (1.0f + expf(-x));
+}
+// 1 - exp(-x), x >= 0: the series where the difference would cancel
+__device__ __forceinline__ float one_minus_exp(float x, float e) {
+    const float s = x * (1.0f + x * (-0.5f + x * (1.0f / 6.0f + x * (-1.0f / 24.0f + x * (1.0f / 120.0f - x * (1.0f / 720.0f))))));
+    return x < 0.3f ? s : 1.0f - e;
+}
+// one token of one channel: S <- a S + g
+template <bool FAST>
+__device__ __forceinline__ void gates(float zr, float zi, float u, float rb, float ib, float decay, float& a, float& g) {
+    const float x = sigmoid_of<FAST>(zr + rb) * decay;                    // -log a
+    a = exp_of<FAST>(-x);
+    g = sqrtf(FAST ? one_minus_exp(2.0f * x, a * a) : -expm1f(-2.0f * x)) * sigmoid_of<FAST>(zi + ib) * u;
+}
+// 0.5 y (1 + tanh z) = y / (1 + exp(-2 z)),  z = sqrt(2 / pi) (y + 0.044715 y^3)
+template <bool FAST> __device__ __forceinline__ float gelu_tanh(float y) {
+    const float z2 = 2.0f * 0.7978845608028654f * (y + 0.044715f * y * y * y);
+    return FAST ? __fdividef(y, 1.0f + __expf(fminf(-z2, 80.0f))) : y / (1.0f + expf(-z2));
+}
+
+struct LruParams {
+    ktk_lru a;
+    ktk_paged t;
+    const float* z;
+    const void *u, *y;
+    int64_t row_stride;
+    const int32_t *new_indptr, *slots;
+    int64_t num_slots, rows;
+    const float *rb, *ib, *decay;
+    float* state;
+    void* out;
+    int32_t* status;
+};
+
+// 16 channels of one sequence: thread (channel, segment) holds 8 consecutive tokens of a tile of 128.
+template <typename T>
+__global__ void __launch_bounds__(kLsThreads, 2) lru_scan_kernel(const LruParams p) {
+    constexpr bool FAST = sizeof(T) == 2;
+    __shared__ float seg_a[kLsSegs][kLsChan + 1], seg_s[kLsSegs][kLsChan + 1], in_s[kLsSegs][kLsChan + 1];
+    Run r;
+    if (!run_of(p.t, p.new_indptr, p.slots, p.num_slots, blockIdx.y, p.status, r)) return;
+    const int bs = p.a.block_stride, width = p.a.blocks * bs;
+    const int tid = threadIdx.x, ch = tid % kLsChan, seg = tid / kLsChan;
+    const int c = blockIdx.x * kLsChan + ch;
+    const bool on = c < width;
+    const int blk = on ? c / bs : 0, cc = on ? c - blk * bs : 0;
+    const float* z = p.z + ((int64_t)blk * p.rows + r.row0) * (2 * bs) + cc;
+    const T* u = (const T*)p.u + r.row0 * width + (on ? c : 0);
+    const T* y = (const T*)p.y + r.row0 * p.row_stride + (on ? c : 0);
+    T* out = (T*)p.out + r.row0 * width + c;
+    const float rb = on ? p.rb[c] : 0.0f, ib = on ? p.ib[c] : 0.0f, decay = on ? p.decay[c] : 0.0f;
+    // a thread of segment s, channel `ch` joins; lane = (channel of the pair, segment): a warp holds two channels
+    const int lane = tid & 31, jch = (tid >> 5) * 2 + (lane >> 4), jseg = lane & 15;
+    const int jc = blockIdx.x * kLsChan + jch;
+    float carry = jc < width && r.base > 0 ? p.state[(int64_t)r.slot * width + jc] : 0.0f;
+
+    float zr[kLsRun], zi[kLsRun];
+    T uu[kLsRun], yy[kLsRun];
+    auto fetch = [&](int tile) {
+#pragma unroll
+        for (int k = 0; k < kLsRun; ++k) {
+            const int i = tile * kLsTile + seg * kLsRun + k;
+            if (on && i < r.n) {
+                zr[k] = __ldcs(z + (int64_t)i * (2 * bs));
+                zi[k] = __ldcs(z + (int64_t)i * (2 * bs) + bs);
+                uu[k] = u[(int64_t)i * width];
+                yy[k] = y[(int64_t)i * p.row_stride];
+            }
+        }
+    };
+    const int tiles = (r.n + kLsTile - 1) / kLsTile;
+    fetch(0);
+    for (int tile = 0; tile < tiles; ++tile) {
+        float a[kLsRun], g[kLsRun], yg[kLsRun], A = 1.0f, S = 0.0f;
+        const int i0 = tile * kLsTile + seg * kLsRun;
+#pragma unroll
+        for (int k = 0; k < kLsRun; ++k) {
+            a[k] = 1.0f;
+            g[k] = yg[k] = 0.0f;
+            if (on && i0 + k < r.n) {
+                gates<FAST>(zr[k], zi[k], to_f32(uu[k]), rb, ib, decay, a[k], g[k]);
+                yg[k] = gelu_tanh<FAST>(to_f32(yy[k]));
+            }
+            A *= a[k];
+            S = fmaf(a[k], S, g[k]);
+        }
+        if (tile + 1 < tiles) fetch(tile + 1);
+        seg_a[seg][ch] = A;
+        seg_s[seg][ch] = S;
+        __syncthreads();
+        float ja = seg_a[jseg][jch], js = seg_s[jseg][jch];
+#pragma unroll
+        for (int o = 1; o < kLsSegs; o <<= 1) {            // inclusive join over the 16 lanes of a channel
+            const float pa = __shfl_up_sync(0xffffffffu, ja, o, kLsSegs), ps = __shfl_up_sync(0xffffffffu, js, o, kLsSegs);
+            if (jseg >= o) { js = fmaf(ja, ps, js); ja *= pa; }
+        }
+        const float end = fmaf(ja, carry, js);             // state behind segment jseg
+        const float before = __shfl_up_sync(0xffffffffu, end, 1, kLsSegs);
+        in_s[jseg][jch] = jseg == 0 ? carry : before;
+        carry = __shfl_sync(0xffffffffu, end, kLsSegs - 1, kLsSegs);
+        __syncthreads();
+        S = in_s[seg][ch];
+#pragma unroll
+        for (int k = 0; k < kLsRun; ++k) {
+            S = fmaf(a[k], S, g[k]);
+            if (on && i0 + k < r.n) out[(int64_t)(i0 + k) * width] = from_f32<T>(S * yg[k]);
+        }
+    }
+    if (jc < width && jseg == 0) p.state[(int64_t)r.slot * width + jc] = carry;
+}
+
+// One token of every sequence: a thread per channel.
+template <typename T>
+__global__ void __launch_bounds__(kLdThreads) lru_step_kernel(const LruParams p) {
+    constexpr bool FAST = sizeof(T) == 2;
+    Run r;
+    if (!run_of(p.t, nullptr, p.slots, p.num_slots, blockIdx.y, p.status, r)) return;
+    const int bs = p.a.block_stride, width = p.a.blocks * bs;
+    const int c = blockIdx.x * kLdThreads + threadIdx.x;
+    if (c >= width) return;
+    const int blk = c / bs, cc = c - blk * bs;
+    const float* z = p.z + ((int64_t)blk * p.rows + r.row0) * (2 * bs) + cc;
+    float* state = p.state + (int64_t)r.slot * width + c;
+    float a, g;
+    gates<FAST>(z[0], z[bs], to_f32(((const T*)p.u)[r.row0 * width + c]), p.rb[c], p.ib[c], p.decay[c], a, g);
+    const float S = fmaf(a, r.base > 0 ? *state : 0.0f, g);
+    *state = S;
+    ((T*)p.out)[r.row0 * width + c] = from_f32<T>(S * gelu_tanh<FAST>(to_f32(((const T*)p.y)[r.row0 * p.row_stride + c])));
+}
+
+static int check_lru(const ktk_lru* a, const ktk_paged* t, const int32_t* new_indptr, int64_t rows, int32_t max_new,
+                     int64_t row_stride, int64_t col, int64_t num_slots, const char* who) {
+    if (a == nullptr || t == nullptr || a->blocks <= 0 || a->block <= 0 || a->block_stride < a->block ||
+        a->block_stride % 8 != 0 || a->taps <= 0 || a->taps > 1024 || (a->dtype != KTK_F32 && a->dtype != KTK_BF16) ||
+        (int64_t)a->blocks * a->block_stride > (1 << 24) || t->page_size <= 0 || t->batch < 0 || t->batch > 65535) {
+        set_error("%s: bad sizes", who);
+        return KTK_ERR_ARG;
+    }
+    const int width = a->blocks * a->block_stride;
+    if (rows < 0 || rows > 2147483647LL || (!new_indptr && rows != t->batch) || (new_indptr && max_new < 0) || row_stride % 8 != 0 ||
+        col % 8 != 0 || col < 0 || col + width > row_stride || num_slots < 0) {
+        set_error("%s: %lld rows for %d sequences, columns %lld of %lld", who, (long long)rows, t->batch, (long long)col,
+                  (long long)row_stride);
+        return KTK_ERR_ARG;
+    }
+    return KTK_OK;
+}
+
+template <typename T>
+static int conv_launch(const void* x, int64_t row_stride, const int32_t* ni, int max_new, const int32_t* slots, int64_t num_slots,
+                       const float* w, const float* b, void* ring, void* u, const ktk_paged& t, const ktk_lru& a,
+                       int32_t* status, cudaStream_t st) {
+    const int width = a.blocks * a.block_stride, chunk = a.taps > kLcChunk ? a.taps : kLcChunk;
+    const int n = ni ? max_new : 1;
+    const dim3 grid((unsigned)((width / 8 + kLcThreads - 1) / kLcThreads), (unsigned)((n + chunk - 1) / chunk), (unsigned)t.batch);
+    if (grid.y > 65535) { set_error("ktk_lru_conv: %d tokens in one call", n); return KTK_ERR_TOO_LARGE; }
+    auto kernel = a.taps == 4 ? lru_conv_kernel<T, 4> : lru_conv_kernel<T, 0>;
+    kernel<<<grid, kLcThreads, 0, st>>>((const T*)x, row_stride, ni, slots, num_slots, w, b, (T*)ring, (T*)u, t, width, a.taps,
+                                        chunk, status);
+    KTK_CUDA_TRY(cudaGetLastError(), "ktk_lru_conv");
+    return KTK_OK;
+}
+
+template <typename T> static int scan_launch(const LruParams& p, cudaStream_t st) {
+    const int width = p.a.blocks * p.a.block_stride;
+    if (p.new_indptr)
+        lru_scan_kernel<T><<<dim3((unsigned)((width + kLsChan - 1) / kLsChan), (unsigned)p.t.batch), kLsThreads, 0, st>>>(p);
+    else
+        lru_step_kernel<T><<<dim3((unsigned)((width + kLdThreads - 1) / kLdThreads), (unsigned)p.t.batch), kLdThreads, 0, st>>>(p);
+    KTK_CUDA_TRY(cudaGetLastError(), "ktk_lru_scan");
+    return KTK_OK;
+}
+
+}  // namespace ktk
+
+using namespace ktk;
+
+extern "C" int ktk_lru_conv(const void* proj, int64_t row_stride, int64_t x_col, const int32_t* new_indptr, int64_t rows,
+                            int32_t max_new, const int32_t* slots, int64_t num_slots, const float* conv_w,
+                            const float* conv_b, void* ring, void* u, const ktk_paged* table, const ktk_lru* shape,
+                            int32_t* status, void* stream) {
+    const char* who = "ktk_lru_conv";
+    const int rc = check_lru(shape, table, new_indptr, rows, max_new, row_stride, x_col, num_slots, who);
+    if (rc != KTK_OK) return rc;
+    if (rows == 0 || max_new == 0) return KTK_OK;
+    if (!proj || !slots || !conv_w || !conv_b || !ring || !u || !table->kv_indptr || !table->kv_last_page_len ||
+        (((uintptr_t)proj | (uintptr_t)conv_w | (uintptr_t)conv_b | (uintptr_t)ring | (uintptr_t)u) & 15u) != 0) {
+        set_error("%s: null or misaligned pointer", who);
+        return KTK_ERR_ARG;
+    }
+    cudaStream_t st = (cudaStream_t)stream;
+    if (shape->dtype == KTK_F32)
+        return conv_launch<float>((const float*)proj + x_col, row_stride, new_indptr, max_new, slots, num_slots, conv_w, conv_b,
+                                  ring, u, *table, *shape, status, st);
+    return conv_launch<__nv_bfloat16>((const __nv_bfloat16*)proj + x_col, row_stride, new_indptr, max_new, slots, num_slots,
+                                      conv_w, conv_b, ring, u, *table, *shape, status, st);
+}
+
+extern "C" int ktk_lru_scan(const float* z, const void* u, const void* proj, int64_t row_stride, int64_t y_col,
+                            const int32_t* new_indptr, int64_t rows, int32_t max_new, const int32_t* slots,
+                            int64_t num_slots, const float* rb, const float* ib, const float* decay, float* state,
+                            void* out, const ktk_paged* table, const ktk_lru* shape, int32_t* status, void* stream) {
+    const char* who = "ktk_lru_scan";
+    const int rc = check_lru(shape, table, new_indptr, rows, max_new, row_stride, y_col, num_slots, who);
+    if (rc != KTK_OK) return rc;
+    if (rows == 0 || max_new == 0) return KTK_OK;
+    if (!z || !u || !proj || !slots || !rb || !ib || !decay || !state || !out || !table->kv_indptr || !table->kv_last_page_len) {
+        set_error("%s: null pointer", who);
+        return KTK_ERR_ARG;
+    }
+    const size_t size = shape->dtype == KTK_F32 ? 4 : 2;
+    const LruParams p{*shape, *table, z, u, (const char*)proj + y_col * size, row_stride, new_indptr, slots, num_slots, rows,
+                      rb, ib, decay, state, out, status};
+    return shape->dtype == KTK_F32 ? scan_launch<float>(p, (cudaStream_t)stream) : scan_launch<__nv_bfloat16>(p, (cudaStream_t)stream);
+}

@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(kMsThreads) moe_simt_kernel(const MoeParams p)
                 const int n = n0 + tx + 16 * j;
                 if (n >= N) continue;
                 float v = acc[0][i][j];
-                if (STAGE == 0) v = v / (1.0f + expf(-v)) * acc[1][i][j];
+                if (STAGE == 0) v = gated<false>(v, acc[1][i][j], p.m.limit, p.m.slope, p.m.shift);
                 else v *= wt[ty + 16 * i];
                 ((T*)p.out)[d * N + n] = from_f32<T>(v);
             }

@@ -2,7 +2,7 @@
 //
 // The weights are the M operand and the routed rows the N operand: D[128 weight rows x N rows] += A[128 x 64] . B^T[64
 // x N].  A work item is one tile of up to 256 rows of an expert and a block of 128 weight rows: stage 0 has the gate
-// and the up row of an inner column side by side, so silu(g) * u needs one exchange between neighbouring lanes.  N
+// and the up row of an inner column side by side, so gating needs one exchange between neighbouring lanes.  N
 // follows the tile's row count, and the ring's stages shrink with the rows a tile can have: a decode step with a few
 // rows per expert keeps many weight tiles in flight and moves little else.  Persistent CTAs; the item list follows
 // from the experts' row counts, which each CTA reads and scans itself.  Roles:
@@ -289,7 +289,7 @@ moe_umma_kernel(const MoeParams p, const int tile_rows, const int cta_rows, cons
                     const float first = odd ? got : v[i], second = odd ? v[i + 1] : got;
                     const int row = c0 + i + odd;
                     if (STAGE == 0) {                        // gate and up of inner column wrow / 2
-                        const float act = __fdividef(first, 1.0f + __expf(-first)) * second;
+                        const float act = gated<true>(first, second, p.m.limit, p.m.slope, p.m.shift);
                         if (row < it.n && wrow < N)
                             out[(int64_t)(plan.first_row[it.e] + it.r0 + row) * p.m.ff_stride + (wrow >> 1)] =
                                 __float2bfloat16_rn(act);

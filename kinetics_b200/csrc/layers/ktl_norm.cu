@@ -13,6 +13,7 @@ struct ResidualNormParams {
     const int64_t* tokens;
     const void* embed;
     int64_t vocab;
+    float embed_scale;
     float* x;
     const void* y;
     int parts;
@@ -96,8 +97,11 @@ __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const Residua
 #pragma unroll
         for (int e = 0; e < 8; ++e) x[i][e] = 0.0f;
         if (k < nvec) {
-            if (p.tokens != nullptr) Vec8<T>::load((const T*)p.embed + tok * p.stride + k * 8, x[i]);
-            else Vec8<float>::load(xrow + k * 8, x[i]);
+            if (p.tokens != nullptr) {
+                Vec8<T>::load((const T*)p.embed + tok * p.stride + k * 8, x[i]);
+#pragma unroll
+                for (int e = 0; e < 8; ++e) x[i][e] *= p.embed_scale;
+            } else Vec8<float>::load(xrow + k * 8, x[i]);
         }
     }
     if (p.y != nullptr) {
@@ -130,7 +134,7 @@ __global__ void __launch_bounds__(kRnThreads) residual_norm_kernel(const Residua
         }
     }
     if (p.h != nullptr) {
-        norm_regs<NV>(x, p.pre_w, p.pre_b, p.eps, p.center != 0, p.cols, nvec, part);
+        if (p.pre_w != nullptr) norm_regs<NV>(x, p.pre_w, p.pre_b, p.eps, p.center != 0, p.cols, nvec, part);
 #pragma unroll
         for (int i = 0; i < NV; ++i) {
             const int k = threadIdx.x + i * blockDim.x;
@@ -157,8 +161,8 @@ static int residual_norm_launch(const ResidualNormParams& p, int64_t rows, cudaS
 
 using namespace ktk;
 
-extern "C" int ktk_residual_norm(const int64_t* tokens, const void* embed, int64_t vocab, float* x, const void* y,
-                                 int32_t parts, const float* post_w, const float* post_b, float mult,
+extern "C" int ktk_residual_norm(const int64_t* tokens, const void* embed, int64_t vocab, float embed_scale, float* x,
+                                 const void* y, int32_t parts, const float* post_w, const float* post_b, float mult,
                                  const float* pre_w, const float* pre_b, void* h, float eps, int32_t center,
                                  int64_t rows, int32_t cols, int32_t stride, int32_t* zero, int32_t zero_n,
                                  int32_t dtype, int32_t* status, void* stream) {
@@ -174,14 +178,14 @@ extern "C" int ktk_residual_norm(const int64_t* tokens, const void* embed, int64
         return KTK_ERR_UNSUPPORTED;
     }
     if (rows == 0) return KTK_OK;
-    if (!x || (tokens && (!embed || vocab <= 0)) || (h && !pre_w) || (!h && !y && !tokens)) {
+    if (!x || (tokens && (!embed || vocab <= 0)) || (!h && !y && !tokens)) {
         set_error("%s: null pointer argument", who);
         return KTK_ERR_ARG;
     }
     const uintptr_t al = (uintptr_t)embed | (uintptr_t)x | (uintptr_t)y | (uintptr_t)post_w | (uintptr_t)post_b |
                          (uintptr_t)pre_w | (uintptr_t)pre_b | (uintptr_t)h;
     if ((al & 15u) != 0) { set_error("%s: pointers must be 16-byte aligned", who); return KTK_ERR_ARG; }
-    const ResidualNormParams p{tokens, embed, vocab, x, y, parts, post_w, post_b, mult, pre_w, pre_b, h, eps,
+    const ResidualNormParams p{tokens, embed, vocab, embed_scale, x, y, parts, post_w, post_b, mult, pre_w, pre_b, h, eps,
                                center, cols, stride, zero, zero ? zero_n : 0, status};
     return dtype == KTK_F32 ? residual_norm_launch<float>(p, rows, (cudaStream_t)stream)
                             : residual_norm_launch<__nv_bfloat16>(p, rows, (cudaStream_t)stream);

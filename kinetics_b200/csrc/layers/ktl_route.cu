@@ -27,12 +27,21 @@ struct RouteParams {
     int64_t rows;
 };
 
-// One warp: the `top` largest of z[0 .. experts) (ties to the lower index), the softmax over them.  z is overwritten.
+// One warp: the `top` largest of z[0 .. experts) (ties to the lower index), weighted by the softmax over them or over all.
+// z is overwritten.
 // ids_s [top], shared memory of the warp: the choice, for the caller.
 __device__ __forceinline__ void pick_experts(const RouteParams& p, float* z, int64_t row, int32_t* ids_s) {
     const int lane = threadIdx.x & 31;
     const int E = p.m.experts, top = p.m.top;
-    float best0 = 0.0f, denom = 0.0f;
+    float best0 = 0.0f, denom = 0.0f, denom_all = 0.0f;
+    if (p.m.scoring == 1) {
+        float mx = -INFINITY;
+        for (int i = lane; i < E; i += 32) mx = fmaxf(mx, z[i]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+        for (int i = lane; i < E; i += 32) denom_all += expf(z[i] - mx);
+        denom_all = warp_sum_f(denom_all);
+    }
     for (int j = 0; j < top; ++j) {
         uint32_t key = 0;
         int e = E - 1;
@@ -55,6 +64,7 @@ __device__ __forceinline__ void pick_experts(const RouteParams& p, float* z, int
         }
         __syncwarp();
     }
+    if (p.m.scoring == 1) denom = denom_all;
     for (int j = lane; j < top; j += 32) p.weights[row * top + j] /= denom;
 }
 
@@ -98,8 +108,8 @@ __global__ void __launch_bounds__(kRtRowThreads) route_row_kernel(const RoutePar
         s0 = warp_sum_f(s0);
         s1 = warp_sum_f(s1);
         if (lane == 0) {
-            rt_z[e0] = s0 + p.b[e0];
-            if (e1 != e0) rt_z[e1] = s1 + p.b[e1];
+            rt_z[e0] = p.b ? s0 + p.b[e0] : s0;
+            if (e1 != e0) rt_z[e1] = p.b ? s1 + p.b[e1] : s1;
         }
     }
     __syncthreads();
@@ -182,7 +192,7 @@ __global__ void __launch_bounds__(kRtThreads) route_mma_kernel(const RouteParams
 #pragma unroll
             for (int x = 0; x < 4; ++x) {
                 const int col = e + (x & 1);
-                rt_z[(16 * i + gid + (x >= 2 ? 8 : 0)) * ld + col] = acc[i][x] + (col < E ? p.b[col] : 0.0f);
+                rt_z[(16 * i + gid + (x >= 2 ? 8 : 0)) * ld + col] = acc[i][x] + (p.b && col < E ? p.b[col] : 0.0f);
             }
         __syncthreads();
     }
@@ -211,7 +221,8 @@ using namespace ktk;
 static int check_moe(const ktk_moe* m, int64_t rows, const char* who) {
     if (m == nullptr || rows < 0 || m->experts <= 0 || m->top <= 0 || m->top > m->experts || m->width <= 0 ||
         m->ff <= 0 || m->width_stride < m->width || m->ff_stride < m->ff || m->width_stride % 8 != 0 ||
-        m->ff_stride % 8 != 0 || (m->dtype != KTK_F32 && m->dtype != KTK_BF16)) {
+        m->ff_stride % 8 != 0 || (m->dtype != KTK_F32 && m->dtype != KTK_BF16) ||
+        m->scoring < 0 || m->scoring > 1 || !(m->limit > 0.0f)) {
         set_error("%s: bad sizes", who);
         return KTK_ERR_ARG;
     }
@@ -229,7 +240,7 @@ extern "C" int ktk_moe_route(const void* h, const void* w, const float* b, int32
     const int rc = check_moe(shape, rows, who);
     if (rc != KTK_OK) return rc;
     if (rows == 0) return KTK_OK;
-    if (!h || !w || !b || !ids || !weights || !counts || !bucket || (((uintptr_t)h | (uintptr_t)w) & 15u) != 0) {
+    if (!h || !w || !ids || !weights || !counts || !bucket || (((uintptr_t)h | (uintptr_t)w) & 15u) != 0) {
         set_error("%s: null or misaligned pointer", who);
         return KTK_ERR_ARG;
     }

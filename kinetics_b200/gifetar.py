@@ -23,9 +23,8 @@ from typing import Optional, Tuple
 
 import torch
 
-from . import layer_ops, ops
-from .layer_cache import LayeredKVManager
-from .layer_ops import AttentionSpec, MoeSpec, pad8
+from .layer_ops import AttentionSpec, MoeSpec
+from .layered_model import LayeredModel, WeightPacker
 
 
 @dataclass(frozen=True)
@@ -81,7 +80,7 @@ def _layer_from(entry: dict, at: int) -> GifetarLayer:
                         temp_every=temp["every"], **extra)
 
 
-class Gifetar:
+class Gifetar(LayeredModel):
     @staticmethod
     def from_config(raw: dict) -> GifetarConfig:
         return GifetarConfig(vocab=raw["vocab"], width=raw["width"], norm_eps=raw["norm"]["eps"],
@@ -90,131 +89,50 @@ class Gifetar:
 
     def __init__(self, config: GifetarConfig, weights, device, dtype=torch.bfloat16):
         """weights: mapping of the checkpoint's tensor names (``checkpoint.Checkpoint``, or a dict)."""
-        if dtype not in (torch.bfloat16, torch.float32):
-            raise TypeError(f"Gifetar runs in bfloat16 or float32, not {dtype}")
-        self.config, self.device, self.dtype = config, torch.device(device), dtype
-        self.width, self.stride = config.width, pad8(config.width)
-        self.eps, self.mult = config.norm_eps, config.residual_mult
-        self.status = ops.new_status(self.device)
-        W, C, S = weights, config.width, self.stride
-        zeros = lambda *shape: torch.zeros(*shape, dtype=dtype, device=self.device)
-
-        def heads(name, groups, size, cols=C):
-            """[groups * size, cols] -> [groups * pad8(size), stride], zeros in the padding."""
-            t = W[name]
-            if tuple(t.shape) != (groups * size, cols):
-                raise ValueError(f"{name}: shape {tuple(t.shape)}, expected {(groups * size, cols)}")
-            out = zeros(groups, pad8(size), pad8(cols))
-            out[:, :size, :cols] = t.view(groups, size, cols)
-            return out.view(groups * pad8(size), pad8(cols))
-
-        def vector(name, groups, size, to=torch.float32):
-            t = W[name]
-            if t.numel() != groups * size:
-                raise ValueError(f"{name}: {t.numel()} values, expected {groups * size}")
-            out = torch.zeros(groups, pad8(size), dtype=to, device=self.device)
-            out[:, :size] = t.view(groups, size)
-            return out.view(-1)
-
-        norm = lambda name: (vector(name, 1, C), vector(name + ".b", 1, C))
-        table = W["embed"]
-        if tuple(table.shape) != (config.vocab, C):
-            raise ValueError(f"embed: shape {tuple(table.shape)}, expected {(config.vocab, C)}")
-        self.embed = zeros(config.vocab, S)
-        self.embed[:, :C] = table
+        super().__init__(config, device, dtype)
+        pack, C = WeightPacker(weights, self.device, dtype), self.width
+        self.mult = config.residual_mult
+        norm = lambda name: (pack.vector(name, 1, C), pack.vector(name + ".b", 1, C))
+        self._load_table(pack)
         self.final_norm = norm("final.norm")
-        self.layers, self.attention_specs = [], []
         for i, l in enumerate(config.layers):
             p, mx = f"l{i}.", f"l{i}.mix."
             H2, G2 = l.heads * 2, l.kv_heads * 2
-            dot = lambda a, b: float((W[mx + a].double() * W[mx + b].double()).sum())
+            dot = lambda a, b: float((pack[mx + a].double() * pack[mx + b].double()).sum())
             lam = math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + l.diff
             spec = l.attention(lam, self.eps)
-            o = W[mx + "o"]
-            if tuple(o.shape) != (C, l.heads * l.vdim):
-                raise ValueError(f"{mx}o: shape {tuple(o.shape)}, expected {(C, l.heads * l.vdim)}")
-            o_pad = zeros(S, l.heads, spec.vdim_stride)
-            o_pad[:C, :, :l.vdim] = o.view(C, l.heads, l.vdim)
             layer = dict(
                 norm1=norm(p + "norm1"), norm1b=norm(p + "norm1b"), spec=spec, moe=l.moe(C),
-                wqkv=torch.cat((heads(mx + "q", H2, l.dim), heads(mx + "k", G2, l.dim),
-                                heads(mx + "v", l.kv_heads, l.vdim))),
-                bqkv=torch.cat((vector(mx + "q.b", H2, l.dim, dtype), vector(mx + "k.b", G2, l.dim, dtype),
-                                vector(mx + "v.b", l.kv_heads, l.vdim, dtype))),
-                wo=o_pad.view(S, l.heads * spec.vdim_stride))
+                wqkv=torch.cat((pack.matrix(mx + "q", (H2, l.dim), C), pack.matrix(mx + "k", (G2, l.dim), C),
+                                pack.matrix(mx + "v", (l.kv_heads, l.vdim), C))),
+                bqkv=torch.cat((pack.vector(mx + "q.b", H2, l.dim, dtype), pack.vector(mx + "k.b", G2, l.dim, dtype),
+                                pack.vector(mx + "v.b", l.kv_heads, l.vdim, dtype))),
+                wo=pack.matrix(mx + "o", C, (l.heads, l.vdim)))
             if layer["moe"] is not None:
-                f, ml = l.ff, p + "mlp."
-                gate_up, down = zeros(l.experts, pad8(f), 2, S), zeros(l.experts, S, pad8(f))
-                for e in range(l.experts):
-                    gate_up[e, :f, 0, :C] = W[f"{ml}e{e}.gate"]
-                    gate_up[e, :f, 1, :C] = W[f"{ml}e{e}.up"]
-                    down[e, :C, :f] = W[f"{ml}e{e}.down"]
-                router = zeros(l.experts, S)
-                router[:, :C] = W[ml + "router"]
-                layer.update(norm2=norm(p + "norm2"), norm2b=norm(p + "norm2b"), router=router,
-                             router_b=W[ml + "router.b"].float().to(self.device), gate_up=gate_up, down=down,
-                             counts=torch.zeros(l.experts, dtype=torch.int32, device=self.device))
+                layer.update(norm2=norm(p + "norm2"), norm2b=norm(p + "norm2b"),
+                             **pack.experts(p + "mlp.", layer["moe"], bias=True))
             self.layers.append(layer)
-            self.attention_specs.append(spec)
+            self.cache_specs.append(spec)
 
-    def new_cache(self, max_batch: int, max_seq_len: int, num_pages: Optional[int] = None, page_size: int = 64,
-                  alias_layers: bool = False) -> LayeredKVManager:
-        return LayeredKVManager(self.attention_specs, max_batch, max_seq_len, self.device, self.dtype, num_pages,
-                                page_size, alias_layers)
-
-    # ---- forward
     def _hidden(self, input_ids, batch_idx, kv, streams=None):
         """The final norm of every row, [rows, stride].  `streams`, a list, receives the residual stream behind every
         layer (a debugging aid)."""
-        bsz, seq_len = input_ids.shape
-        if bsz != 1 and seq_len != 1:
-            raise ValueError(f"one sequence, or one token of each: input shape {tuple(input_ids.shape)}")
-        rows, S, dev = bsz * seq_len, self.stride, self.device
-        x = torch.empty(rows, S, dtype=torch.float32, device=dev)
-        h = torch.empty(rows, S, dtype=self.dtype, device=dev)
-        step = lambda **kw: layer_ops.residual_norm(x, h, self.width, self.eps, status=self.status, **kw)
+        x, h, step = self._stream(input_ids)
         step(tokens=input_ids.reshape(-1).to(torch.int64).contiguous(), embed=self.embed,
              pre=self.layers[0]["norm1"] if self.layers else self.final_norm)
         for i, L in enumerate(self.layers):
             after = self.layers[i + 1]["norm1"] if i + 1 < len(self.layers) else self.final_norm
             proj = torch.addmm(L["bqkv"], h, L["wqkv"].t())
-            attn = kv.attend(proj, i, batch_idx, seq_len)
+            attn = kv.attend(proj, i, batch_idx, input_ids.shape[1])
             y = torch.mm(attn, L["wo"].t())
             if L["moe"] is None:
                 step(y=y, post=L["norm1b"], mult=self.mult, pre=after)
             else:
                 step(y=y, post=L["norm1b"], mult=self.mult, pre=L["norm2"], zero=L["counts"])
-                routing = layer_ops.moe_route(h, L["router"], L["router_b"], L["moe"], L["counts"])
-                y = layer_ops.moe_experts(h, L["gate_up"], L["down"], routing, L["moe"], status=self.status)
-                step(y=y, parts=L["moe"].top, post=L["norm2b"], mult=self.mult, pre=after)
+                step(y=self._experts(h, L), parts=L["moe"].top, post=L["norm2b"], mult=self.mult, pre=after)
             if streams is not None:
                 streams.append(x[:, :self.width].clone())
         return h
-
-    def _logits(self, h):
-        if self.dtype == torch.float32:
-            return torch.mm(h, self.embed.t())
-        return torch.mm(h, self.embed.t(), out_dtype=torch.float32)
-
-    @torch.no_grad()
-    def inference(self, input_ids, position_ids, batch_idx, kv, rows=None):
-        """input_ids [B, S] (one sequence's next S tokens, or one token of B sequences) -> fp32 logits [B, S, V].
-        Positions are those of the cache (`position_ids` is what Engine passes to every model).  rows: project only
-        these of the S tokens of a sequence, [1, len(rows), V]."""
-        h = self._hidden(input_ids, batch_idx, kv)
-        if rows is not None:
-            h = h[torch.as_tensor(rows, dtype=torch.int64, device=h.device)]
-            return self._logits(h).unsqueeze(0)
-        return self._logits(h).view(*input_ids.shape, -1)
-
-    @torch.no_grad()
-    def next_tokens(self, input_ids, position_ids, batch_idx, kv, last_only: bool = False):
-        """Greedy tokens of the rows (last_only: of the last row, a prompt's)."""
-        h = self._hidden(input_ids, batch_idx, kv)
-        return self._logits(h[-1:] if last_only else h).argmax(dim=-1)
-
-    def check_status(self):
-        ops.raise_on_status(self.status)
 
 
 def random_weights(config: GifetarConfig, seed: int = 0, device="cpu", dtype=torch.bfloat16) -> dict:

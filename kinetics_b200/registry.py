@@ -13,8 +13,9 @@ import torch
 
 from .checkpoint import Checkpoint
 from .gifetar import Gifetar
+from .munadra import Munadra
 
-MODELS = {"Gifetar": Gifetar}
+MODELS = {"Gifetar": Gifetar, "Munadra": Munadra}
 
 
 def model_class(config: dict):

@@ -229,15 +229,15 @@ def test_header_and_binding_of_the_layer_library_agree():
     one, null = ctypes.c_void_p(16), ctypes.c_void_p(0)
     a = _lib.Attn(4, 3, 2, 8, 8, 8, 8, 1, 1.0, 0.0, 0.0, 1.0, 0.0, 0.0, 1.0)
     t = _lib.Paged(16, 16, 16, 1, 16, 4)
-    call = lambda: lib.ktk_paged_attention(one, 64, null, 1, 1, one, one, ctypes.byref(t), one, null, 0, 1, 0,
-                                           ctypes.byref(a), null, null)
+    call = lambda: lib.ktk_paged_attention(one, 64, null, 1, 1, one, one, ctypes.byref(t), null, null, 0, one,
+                                           null, 0, 1, 0, ctypes.byref(a), null, null)
     assert call() == -1                                    # 4 heads over 3 kv heads
     a.kv_heads = 2
     t.page_size = 24
     assert call() == -2 and b"page_size" in lib.ktk_last_error()
     m = _lib.Moe(4, 5, 8, 8, 8, 8, 1, 0)
     assert lib.ktk_moe_route(one, one, one, one, one, one, one, 1, ctypes.byref(m), 0, null) == -1
-    assert lib.ktk_residual_norm(null, null, 0, one, null, 1, null, null, 1.0, null, null, null, 1e-6, 1, 1, 12, 12, null,
+    assert lib.ktk_residual_norm(null, null, 0, 1.0, one, null, 1, null, null, 1.0, null, null, null, 1e-6, 1, 1, 12, 12, null,
                                  0, 1, null, null) == -1   # a stride of 12
 
 
