@@ -80,11 +80,12 @@ KTK_API int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col, i
  * Causal attention of new tokens (already in their pages) over their sequence.
  * q [rows, q_stride]: heads * maps * dim_stride columns, head by head and map by map; o [rows, heads * vdim_stride].
  * variant: KTK_VARIANT_AUTO, _SIMT (any size, fp32 math), _MMA (bf16, one row per sequence), _UMMA (bf16 on tcgen05).
- * splits: parts that a sequence's keys are cut into where new_indptr is null (0: policy).
+ * splits: parts that a sequence's keys are cut into (0: policy); with new_indptr only where values lie in the keys.
+ * The policy's new_rows: 0 for one row per sequence, else the rows of each.
  * sink fp32 [heads] (nullable, maps = 1): exp(sink) joins each row's denominator, without key, value or scale.
  * gate (nullable, maps = 1), in `dtype`: head h of row r is multiplied by sigmoid(gate[r * gate_stride + h]).
  */
-KTK_API int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int64_t max_keys);
+KTK_API int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int32_t new_rows, int64_t max_keys);
 KTK_API size_t ktk_paged_attention_workspace(const ktk_attn* shape, int64_t rows, int32_t splits);
 KTK_API int ktk_paged_attention(const void* q, int64_t q_stride, const int32_t* new_indptr, int64_t rows,
                                 int32_t max_new, const void* k_pages, const void* v_pages, const ktk_paged* table,

@@ -165,7 +165,7 @@ _LAYER_SIGNATURES = {
                                     _i32p, c_int32, c_int32, _i32p, c_void_p]),
     "ktk_kv_append": (c_int32, [c_void_p, c_int64, c_int64, c_int64, _i32p, c_int64, c_void_p, c_void_p,
                                 POINTER(Paged), POINTER(Attn), _i32p, c_void_p]),
-    "ktk_paged_attention_splits": (c_int32, [POINTER(Attn), c_int32, c_int64]),
+    "ktk_paged_attention_splits": (c_int32, [POINTER(Attn), c_int32, c_int32, c_int64]),
     "ktk_paged_attention_workspace": (c_size_t, [POINTER(Attn), c_int64, c_int32]),
     "ktk_paged_attention": (c_int32, [c_void_p, c_int64, _i32p, c_int64, c_int32, c_void_p, c_void_p, POINTER(Paged),
                                       c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_size_t, c_int32, c_int32, POINTER(Attn), _i32p, c_void_p]),

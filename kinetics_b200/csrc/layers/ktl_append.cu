@@ -80,11 +80,14 @@ extern "C" int ktk_kv_append(const void* proj, int64_t row_stride, int64_t k_col
                                               *table, *shape, status, st);
 }
 
-extern "C" int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int64_t max_keys) {
+extern "C" int32_t ktk_paged_attention_splits(const ktk_attn* shape, int32_t batch, int32_t new_rows, int64_t max_keys) {
+    if (attn_shared_supported(*shape)) return attn_shared_splits(*shape, batch, new_rows, max_keys);
+    if (new_rows > 0) return 1;
     return attn_decode_supported(*shape) ? attn_decode_splits(*shape, batch, max_keys) : 1;
 }
 
 extern "C" size_t ktk_paged_attention_workspace(const ktk_attn* shape, int64_t rows, int32_t splits) {
+    if (attn_shared_supported(*shape)) return attn_shared_workspace(*shape, rows, splits);
     return attn_decode_supported(*shape) ? attn_decode_workspace(*shape, rows, splits) : 0;
 }
 
@@ -117,10 +120,19 @@ extern "C" int ktk_paged_attention(const void* q, int64_t q_stride, const int32_
     AttnParams p{*shape, *table, q, q_stride, new_indptr, rows, max_new, k_pages, v_pages, sink, gate, gate_stride, o,
                  (float*)workspace, splits, status};
     const bool can_decode = !new_indptr && attn_decode_supported(*shape);
-    const bool can_umma = new_indptr && attn_umma_supported(*shape);
-    if ((variant == KTK_VARIANT_MMA && !can_decode) || (variant == KTK_VARIANT_UMMA && !can_umma)) {
+    const bool can_umma = new_indptr && attn_umma_supported(*shape), can_shared = attn_shared_supported(*shape);
+    if ((variant == KTK_VARIANT_MMA && !can_decode) || (variant == KTK_VARIANT_UMMA && !can_umma && !can_shared)) {
         set_error("%s: variant %d is not built for this case", who, variant);
         return KTK_ERR_UNSUPPORTED;
+    }
+    if (variant != KTK_VARIANT_SIMT && can_shared) {
+        if (p.splits <= 0) p.splits = attn_shared_splits(*shape, table->batch, new_indptr ? max_new : 0, 1 << 20);
+        const size_t need = attn_shared_workspace(*shape, rows, p.splits);
+        if (need && (!workspace || workspace_bytes < need)) {
+            set_error("%s: workspace of %zu bytes needed, got %zu", who, need, workspace ? workspace_bytes : (size_t)0);
+            return KTK_ERR_WORKSPACE;
+        }
+        return launch_attn_shared(p, (cudaStream_t)stream);
     }
     if (variant != KTK_VARIANT_SIMT && can_umma) return launch_attn_umma(p, (cudaStream_t)stream);
     if (variant != KTK_VARIANT_SIMT && can_decode) {

@@ -379,7 +379,7 @@ __global__ void __launch_bounds__(128) attn_combine_kernel(const AttnParams p, i
 }
 
 bool attn_decode_supported(const ktk_attn& a) {
-    return a.dtype == KTK_BF16 && a.maps == 2 && a.dim_stride <= 128 && a.vdim_stride <= 128;
+    return a.dtype == KTK_BF16 && a.maps == 2 && a.v_row_stride == 0 && a.dim_stride <= 128 && a.vdim_stride <= 128;
 }
 
 static int64_t decode_units(const ktk_attn& a, int64_t batch) {
@@ -388,21 +388,8 @@ static int64_t decode_units(const ktk_attn& a, int64_t batch) {
 }
 
 int32_t attn_decode_splits(const ktk_attn& a, int batch, int64_t max_keys) {
-    const int64_t units = decode_units(a, batch), resident = (int64_t)sm_count() * 3;
-    if (units <= 0) return 1;
-    int64_t most = (max_keys + kAdMinKeys - 1) / kAdMinKeys;
-    if (most > kAdMaxSplits) most = kAdMaxSplits;
-    // two to eight rounds of CTAs; among those the count that leaves the last round fullest
-    int64_t lo = (2 * resident + units - 1) / units, hi = (8 * resident + units - 1) / units, best = 1;
-    if (lo > most) lo = most;
-    if (hi > most) hi = most;
-    double best_fill = 0.0;
-    for (int64_t s = lo < 1 ? 1 : lo; s <= hi; ++s) {
-        const int64_t ctas = units * s, rounds = (ctas + resident - 1) / resident;
-        const double fill = (double)ctas / (double)(rounds * resident);
-        if (fill > best_fill + 0.01) { best_fill = fill; best = s; }
-    }
-    return (int32_t)best;
+    return fill_rounds(decode_units(a, batch), (int64_t)sm_count() * 3, 2, 8, (max_keys + kAdMinKeys - 1) / kAdMinKeys,
+                       kAdMaxSplits);
 }
 
 size_t attn_decode_workspace(const ktk_attn& a, int64_t rows, int splits) {

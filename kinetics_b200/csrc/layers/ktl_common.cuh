@@ -115,6 +115,23 @@ inline ktk_attn latent_rows(const ktk_latent& a) {
     return r;
 }
 
+// splits of each of `units` pieces of work: between `lo_rounds` and `hi_rounds` rounds of `resident` CTAs, and among those
+// the count that leaves the last round fullest
+inline int32_t fill_rounds(int64_t units, int64_t resident, int lo_rounds, int hi_rounds, int64_t most, int64_t cap) {
+    if (units <= 0) return 1;
+    if (most > cap) most = cap;
+    int64_t lo = (lo_rounds * resident + units - 1) / units, hi = (hi_rounds * resident + units - 1) / units, best = 1;
+    if (lo > most) lo = most;
+    if (hi > most) hi = most;
+    double best_fill = 0.0;
+    for (int64_t s = lo < 1 ? 1 : lo; s <= hi; ++s) {
+        const int64_t ctas = units * s, rounds = (ctas + resident - 1) / resident;
+        const double fill = (double)ctas / (double)(rounds * resident);
+        if (fill > best_fill + 0.01) { best_fill = fill; best = s; }
+    }
+    return (int32_t)best;
+}
+
 int launch_attn_simt(const AttnParams& p, cudaStream_t st);
 bool attn_decode_supported(const ktk_attn& a);
 int32_t attn_decode_splits(const ktk_attn& a, int batch, int64_t max_keys);
@@ -122,6 +139,10 @@ size_t attn_decode_workspace(const ktk_attn& a, int64_t rows, int splits);
 int make_cache_maps(const AttnParams& p, struct CUtensorMap_st* k_map, struct CUtensorMap_st* v_map, unsigned box_rows, const char* who);
 int launch_attn_decode(const AttnParams& p, cudaStream_t st);
 bool attn_umma_supported(const ktk_attn& a);
+bool attn_shared_supported(const ktk_attn& a);
+int32_t attn_shared_splits(const ktk_attn& a, int batch, int new_rows, int64_t max_keys);
+size_t attn_shared_workspace(const ktk_attn& a, int64_t rows, int splits);
+int launch_attn_shared(const AttnParams& p, cudaStream_t st);
 int launch_attn_umma(const AttnParams& p, cudaStream_t st);
 
 // ---- experts ------------------------------------------------------------------------------------------------

@@ -118,12 +118,11 @@ class LayeredKVManager(PooledTable):
         return LayerStep(table, new_indptr, slots_dev, len(slots), int(self._host_len[layer_idx][slots].max()))
 
     def _attention(self, q, k, v, step: LayerStep, spec: layer_ops.AttentionSpec, seq_len: int, **kw) -> torch.Tensor:
-        splits = 1
-        if step.new_indptr is None:
-            splits = layer_ops.attention_splits(spec, step.sequences, 1 << (step.longest - 1).bit_length(), self.dtype)
-            need = layer_ops.attention_workspace(spec, step.sequences, splits, self.dtype)
-            if need and (self._workspace is None or self._workspace.numel() < need):
-                self._workspace = torch.empty(need, dtype=torch.uint8, device=self.device)
+        splits = layer_ops.attention_splits(spec, step.sequences, 1 << (step.longest - 1).bit_length(), self.dtype,
+                                            0 if step.new_indptr is None else seq_len)
+        need = layer_ops.attention_workspace(spec, q.shape[0], splits, self.dtype)
+        if need and (self._workspace is None or self._workspace.numel() < need):
+            self._workspace = torch.empty(need, dtype=torch.uint8, device=self.device)
         return layer_ops.paged_attention(q, k, v, step.table, spec, step.new_indptr, seq_len, splits, self._workspace,
                                          status=self.status, **kw)
 

@@ -263,9 +263,9 @@ def kv_append(proj, k_col: int, v_col: int, k_pages, v_pages, table: PageTable, 
     _launched()
 
 
-def attention_splits(spec: AttentionSpec, batch: int, max_keys: int, dtype) -> int:
+def attention_splits(spec: AttentionSpec, batch: int, max_keys: int, dtype, new_rows: int = 0) -> int:
     a = spec.c(_lib.KTK_BF16 if dtype == torch.bfloat16 else _lib.KTK_F32)
-    return int(_lib.load_layers().ktk_paged_attention_splits(ctypes.byref(a), batch, max_keys))
+    return int(_lib.load_layers().ktk_paged_attention_splits(ctypes.byref(a), batch, new_rows, max_keys))
 
 
 def attention_workspace(spec: AttentionSpec, rows: int, splits: int, dtype) -> int:
@@ -291,7 +291,7 @@ def paged_attention(proj, k_pages, v_pages, table: PageTable, spec: AttentionSpe
     rows = proj.shape[0]
     if out is None:
         out = torch.empty(rows, spec.o_cols, dtype=proj.dtype, device=proj.device)
-    if new_indptr is None and workspace is None:
+    if splits > 1 and workspace is None:
         need = attention_workspace(spec, rows, splits, proj.dtype)
         if need:
             workspace = torch.empty(need, dtype=torch.uint8, device=proj.device)
@@ -300,7 +300,7 @@ def paged_attention(proj, k_pages, v_pages, table: PageTable, spec: AttentionSpe
         _ptr(proj), proj.shape[1], _ptr(new_indptr), rows, max_new, _ptr(k_pages), _ptr(v_pages), ctypes.byref(t),
         _ptr(sink), None if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0), _ptr(out),
         _ptr(workspace), wsb, splits, variant, ctypes.byref(a), _ptr(status), _stream()))
-    _launched(2 if new_indptr is None and splits > 1 else 1)
+    _launched(2 if splits > 1 else 1)
     return out
 
 

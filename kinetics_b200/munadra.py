@@ -215,3 +215,54 @@ class Munadra(LayeredModel):
         if self.config.logit_scale > 0:                  # scale and softcap keep the order
             return self._project(h).argmax(dim=-1)
         return self._logits(h).argmax(dim=-1)
+
+
+def random_weights(config: MunadraConfig, seed: int = 0, device="cpu", dtype=torch.bfloat16) -> dict:
+    """Random tensors under the checkpoint's names (tests and benchmarks): projections with variance 1 / fan-in, norm
+    weights around zero, decays spread over short and long memories."""
+    g = torch.Generator(device=device).manual_seed(seed)
+    C, W = config.width, {}
+
+    def put(name, *shape, std=None, mean=0.0):
+        std = 1.0 / math.sqrt(shape[-1]) if std is None else std
+        W[name] = (torch.randn(*shape, generator=g, device=device) * std + mean).to(dtype)
+
+    put("embed", config.vocab, C, std=1.0)
+    for i, l in enumerate(config.layers):
+        p, mx, s = f"l{i}.", f"l{i}.mix.", l.mixer
+        for n in ("norm1",) + (("norm2",) if l.ff else ()):
+            put(p + n, C, std=0.1)
+        if isinstance(s, LatentSpec):
+            put(mx + "q", s.heads * (s.dim + s.rot_dim), C)
+            if s.kv_from is None:
+                put(mx + "dkv", s.rank + s.rot_dim, C)
+                put(mx + "dkv.norm", s.rank, std=0.1, mean=1.0)
+            put(mx + "uk", s.heads * s.dim, s.rank)
+            put(mx + "uv", s.heads * s.vdim, s.rank)
+            put(mx + "sink", s.heads, std=1.0)
+            put(mx + "g", s.heads, C)
+            put(mx + "o", C, s.heads * s.vdim)
+        else:
+            n = s.blocks * s.block
+            for b in ("y", "x"):
+                put(mx + b, n, C)
+                put(f"{mx}{b}.b", n, std=0.1)
+            put(mx + "conv", n, s.taps)
+            put(mx + "conv.b", n, std=0.1)
+            for r in ("ra", "ri"):
+                put(mx + r, s.blocks, s.block, s.block)
+                put(f"{mx}{r}.b", s.blocks, s.block, std=0.5)
+            put(mx + "lam", n, std=1.5, mean=-4.0)
+            put(mx + "o", C, n)
+        if l.experts:
+            for e in range(l.experts):
+                put(f"{p}mlp.e{e}.gate", l.ff, C)
+                put(f"{p}mlp.e{e}.up", l.ff, C)
+                put(f"{p}mlp.e{e}.down", C, l.ff)
+            put(p + "mlp.router", l.experts, C)
+        elif l.ff:
+            put(p + "mlp.gate", l.ff, C)
+            put(p + "mlp.up", l.ff, C)
+            put(p + "mlp.down", C, l.ff)
+    put("final.norm", C, std=0.1)
+    return W
