@@ -120,6 +120,21 @@ KTK_API int ktk_latent_append(void* proj, int64_t row_stride, int64_t q_col, int
                               int64_t rows, const float* norm_w, const float* freqs, void* q_out, void* pages,
                               const ktk_paged* table, const ktk_latent* shape, int32_t* status, void* stream);
 
+/*
+ * The newest `rows` of a sequence of `total` tokens over keys and values expanded from its latents:
+ *   q: rows of [dim_stride | rot_stride] per head, rotated;  kv [total, heads * dim_stride | heads * vdim_stride], the
+ *   unrotated keys and the values of every head;  latents [total, rank_stride + rot_stride] (ktk_gather_rows), whose
+ *   rotated keys all heads share;  sink, gate as in ktk_paged_attention;  o [rows, heads * vdim_stride].
+ * bf16; ktk_expanded_attention_supported tells whether it is built for the sizes.
+ */
+KTK_API int ktk_expanded_attention_supported(const ktk_latent* shape);
+KTK_API int ktk_expanded_attention(const void* q, int64_t q_stride, int64_t rows, int64_t total, const void* kv,
+                                   const void* latents, const float* sink, const void* gate, int64_t gate_stride, void* o,
+                                   const ktk_latent* shape, int32_t* status, void* stream);
+/* The first `total` token rows of a table's only sequence out of pages [num_pages, page_size, row_bytes], in order. */
+KTK_API int ktk_gather_rows(const void* pages, void* out, int64_t total, int32_t row_bytes, const ktk_paged* table,
+                            int32_t* status, void* stream);
+
 /* Linear recurrence with real gates, per channel (blocks of block_stride channels, the first `block` of them real):
  *   u = conv_b + sum_k conv_w[k] x_(t - taps + 1 + k)                     causal, zeros before the sequence
  *   r = sigmoid(zr + rb), i = sigmoid(zi + ib)                            zr, zi: block-diagonal products of u

@@ -171,6 +171,10 @@ _LAYER_SIGNATURES = {
                                       c_void_p, c_void_p, c_int64, c_void_p, c_void_p, c_size_t, c_int32, c_int32, POINTER(Attn), _i32p, c_void_p]),
     "ktk_latent_append": (c_int32, [c_void_p, c_int64, c_int64, c_int64, _i32p, c_int64, c_void_p, c_void_p, c_void_p,
                                     c_void_p, POINTER(Paged), POINTER(Latent), _i32p, c_void_p]),
+    "ktk_expanded_attention_supported": (c_int32, [POINTER(Latent)]),
+    "ktk_expanded_attention": (c_int32, [c_void_p, c_int64, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_void_p,
+                                         c_int64, c_void_p, POINTER(Latent), _i32p, c_void_p]),
+    "ktk_gather_rows": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, POINTER(Paged), _i32p, c_void_p]),
     "ktk_lru_conv": (c_int32, [c_void_p, c_int64, c_int64, _i32p, c_int64, c_int32, _i32p, c_int64, c_void_p, c_void_p,
                                c_void_p, c_void_p, POINTER(Paged), POINTER(Lru), _i32p, c_void_p]),
     "ktk_lru_scan": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_int64, _i32p, c_int64, c_int32, _i32p, c_int64,

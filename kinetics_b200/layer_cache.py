@@ -23,6 +23,9 @@ from . import layer_ops, ops
 from .engine import PooledTable
 
 
+EXPAND_ROWS = 64        # from this many new tokens on, keys and values are expanded from the latents
+
+
 @dataclass
 class LatentWeights:
     """What a latent-attention layer brings to the manager: expansions of the latent to every head's keys
@@ -139,13 +142,20 @@ class LayeredKVManager(PooledTable):
     def attend_latent(self, proj: torch.Tensor, layer_idx: int, batch_idx: torch.Tensor, seq_len: int,
                       w: LatentWeights) -> torch.Tensor:
         """proj [rows, q | latent, rotated key | gates]: appends the latents (unless the layer reads another's), returns
-        the gated attention output [rows, heads * vdim].  The queries take the key expansion, q uk, and the heads' values
-        are expanded behind the attention: per token only the latent row is read."""
+        the gated attention output [rows, heads * vdim].  A decode step and a short portion: the queries take the key
+        expansion, q uk, and the heads' values are expanded behind the attention, so that per token only the latent row is
+        read.  A long portion: keys and values of the whole sequence are expanded first, which is less arithmetic per
+        query."""
         spec = self.specs[layer_idx]
         step = self._step_of(layer_idx, batch_idx, seq_len)
         rows, H, pages = proj.shape[0], spec.heads, self.k_pages[layer_idx]
         gate = proj[:, spec.gate_col:]
         dim, rank, vdim = w.uk.shape[1], w.uk.shape[2], w.uv.shape[1]
+        if rows >= EXPAND_ROWS and step.new_indptr is not None and layer_ops.expanded_supported(spec, self.dtype):
+            layer_ops.latent_append(proj, spec, step.table, pages, w.norm, w.freqs, step.new_indptr, status=self.status)
+            latents = layer_ops.gather_rows(pages, step.table, step.longest, status=self.status)
+            kv = torch.mm(latents[:, :rank], w.ukv.t())
+            return layer_ops.expanded_attention(proj, kv, latents, spec, w.sink, gate, status=self.status)
         q = torch.empty(rows, H, spec.row_cols, dtype=proj.dtype, device=proj.device)
         layer_ops.latent_append(proj, spec, step.table, pages, w.norm, w.freqs, step.new_indptr, q, status=self.status)
         heads = proj[:, :spec.q_cols].view(rows, H, -1)

@@ -393,6 +393,40 @@ def latent_append(proj, spec: LatentSpec, table: PageTable, pages, norm_w, freqs
     _launched()
 
 
+def gather_rows(pages, table: PageTable, total: int, status=None):
+    """The first `total` rows of the table's only sequence, in order: pages [pages, 1, page_size, cols] -> [total, cols]."""
+    _cuda(pages, status)
+    out = torch.empty(total, pages.shape[-1], dtype=pages.dtype, device=pages.device)
+    t = table.c()
+    check_layers(_lib.load_layers().ktk_gather_rows(_ptr(pages), _ptr(out), total, pages.shape[-1] * pages.element_size(),
+                                                    ctypes.byref(t), _ptr(status), _stream()))
+    _launched()
+    return out
+
+
+def expanded_supported(spec: LatentSpec, dtype) -> bool:
+    a = spec.c(_lib.KTK_BF16 if dtype == torch.bfloat16 else _lib.KTK_F32)
+    return bool(_lib.load_layers().ktk_expanded_attention_supported(ctypes.byref(a)))
+
+
+def expanded_attention(proj, kv, latents, spec: LatentSpec, sink=None, gate=None, status=None):
+    """The newest rows of a sequence (proj, whose first columns are the rotated queries) over kv [total, keys of all heads |
+    values of all heads], expanded from latents [total, row_cols] -> [rows, heads * pad8(vdim)]."""
+    _cuda(proj, kv, latents, sink, status)
+    rows, total, H = proj.shape[0], latents.shape[0], spec.heads
+    if tuple(kv.shape) != (total, H * (pad8(spec.dim) + pad8(spec.vdim))) or latents.shape[1] != spec.row_cols or \
+            any(t.dtype != torch.bfloat16 for t in (proj, kv, latents)):
+        raise ValueError(f"expanded_attention: shapes {tuple(kv.shape)}, {tuple(latents.shape)} do not fit {spec}")
+    out = torch.empty(rows, H * pad8(spec.vdim), dtype=proj.dtype, device=proj.device)
+    a = spec.c(_lib.KTK_BF16)
+    check_layers(_lib.load_layers().ktk_expanded_attention(
+        _ptr(proj), proj.stride(0), rows, total, _ptr(kv), _ptr(latents), _ptr(sink),
+        None if gate is None else gate.data_ptr(), 0 if gate is None else gate.stride(0), _ptr(out), ctypes.byref(a),
+        _ptr(status), _stream()))
+    _launched()
+    return out
+
+
 def lru_conv(proj, spec: LruSpec, table: PageTable, slots, conv_w, conv_b, ring, new_indptr=None, max_new: int = 1,
              status=None):
     """The causal convolution of the x columns of proj [rows, 2 * cols] -> u [rows, cols]; updates the ring

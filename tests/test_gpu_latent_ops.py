@@ -85,3 +85,95 @@ def test_sinks_of_every_size(cuda_device):
                 want = plain_rows(q.to(BF).double(), rows.to(BF).double(), vdim, spec.scale, sink.double(),
                                   torch.zeros(1, heads).double(), n - 1)
                 assert (got - want).abs().max() < 2e-2 * max(rms(want), 1e-3), (splits, sink[0])
+
+
+# heads, dim, rot_dim, vdim
+EXPANDED = [(4, 128, 64, 128), (3, 32, 32, 32), (2, 40, 8, 72), (1, 192, 64, 128), (5, 64, 128, 16), (2, 24, 16, 100)]
+
+
+@pytest.mark.parametrize("heads,dim,rot_dim,vdim", EXPANDED)
+def test_expanded_attention(cuda_device, heads, dim, rot_dim, vdim):
+    from kinetics_b200 import layer_ops as lo, ops
+    from kinetics_b200.layer_ops import LatentSpec, Rotation, pad8
+    dev, rank = cuda_device, 48
+    spec = LatentSpec(heads, dim, rot_dim, vdim, rank, 1.2 / (dim + rot_dim) ** 0.5, Rotation(rot_dim, 1e4))
+    d, r, v, R = pad8(dim), pad8(rot_dim), pad8(vdim), pad8(rank)
+    for seed, (total, n) in enumerate([(1, 1), (64, 64), (65, 2), (128, 128), (129, 129), (300, 257), (700, 130), (513, 513)]):
+        g = torch.Generator().manual_seed(seed)
+        first = total - n
+        edges = [0, 1, 63, 64, 65, 127, 128, first - 1, first, first + 1, total // 2, total - 2, total - 1]
+        q, k = pointed_rows(total, first, heads, dim + rot_dim, edges, seed, strength=6.0)
+        keys = k[:, None, :dim] + 0.1 * torch.randn(total, heads, dim, generator=g)
+        values = torch.randn(total, heads, vdim, generator=g)
+        sink, gate = torch.linspace(-4, 6, heads), torch.randn(n, heads, generator=g)
+        proj = torch.zeros(n, spec.proj_cols)
+        qp = proj[:, :spec.q_cols].view(n, heads, d + r)
+        qp[:, :, :dim], qp[:, :, d:d + rot_dim] = q[..., :dim], q[..., dim:]
+        proj[:, spec.gate_col:spec.gate_col + heads] = gate
+        kv = torch.zeros(total, heads * (d + v))
+        kv[:, :heads * d].view(total, heads, d)[:, :, :dim] = keys
+        kv[:, heads * d:].view(total, heads, v)[:, :, :vdim] = values
+        lat = torch.full((total, R + r), float("nan"))
+        lat[:, R:] = 0.0
+        lat[:, R:R + rot_dim] = k[:, dim:]
+        put = lambda t: t.to(BF).to(dev)
+        proj, status = put(proj), ops.new_status(dev)
+        got = lo.expanded_attention(proj, put(kv), put(lat), spec, sink.to(dev), proj[:, spec.gate_col:], status)
+        ops.raise_on_status(status)
+        got = got.view(n, heads, v).double().cpu()
+        r64 = lambda t: t.to(BF).double()
+        for h in range(heads):
+            s = (r64(q[:, h, :dim]) @ r64(keys[:, h]).t() + r64(q[:, h, dim:]) @ r64(k[:, dim:]).t()) * spec.scale
+            want = plain.sigmoid(r64(gate[:, h:h + 1])) * (plain.sink_softmax(s, sink[h].double(), first) @ r64(values[:, h]))
+            err = (got[:, h, :vdim] - want).pow(2).mean(-1).sqrt() / rms(want)
+            assert err.max() < 3e-2, (total, n, h, float(err.max()))
+        assert (got[:, :, vdim:] == 0).all()
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_append_rotates_and_normalises(cuda_device, dtype):
+    from kinetics_b200 import layer_ops as lo, ops
+    from kinetics_b200.layer_ops import LatentSpec, Rotation, pad8
+    dev = cuda_device
+    for seed, (heads, dim, rot_dim, rank, ps, lens, new, scaling) in enumerate([
+            (3, 24, 16, 40, 16, [200], 37, dict(factor=4.0, original=32, fast=6.0, slow=0.5, scaled=True)),
+            (2, 20, 10, 36, 64, [1, 70, 64], None, {}), (1, 8, 2, 130, 32, [9], 9, {}),
+            (5, 128, 64, 512, 64, [5000, 3], None, dict(factor=8.0, original=512, fast=32.0, slow=1.0, scaled=True))]):
+        g = torch.Generator().manual_seed(seed)
+        rotation = Rotation(rot_dim, 3000.0, **scaling)
+        raw = {"dims": rot_dim, "base": 3000.0}
+        if scaling:
+            raw["scaling"] = {k: v for k, v in scaling.items() if k != "scaled"}
+        spec = LatentSpec(heads, dim, rot_dim, 8, rank, 1.0, rotation, eps=1e-3)
+        d, r, R, rows = pad8(dim), pad8(rot_dim), pad8(rank), new or len(lens)
+        q, kv = torch.randn(rows, heads, dim + rot_dim, generator=g), 3 * torch.randn(rows, rank + rot_dim, generator=g)
+        w = torch.randn(rank, generator=g)
+        proj = torch.zeros(rows, spec.proj_cols)
+        qp = proj[:, :spec.q_cols].view(rows, heads, d + r)
+        qp[..., :dim], qp[..., d:d + rot_dim] = q[..., :dim], q[..., dim:]
+        proj[:, spec.q_cols:spec.q_cols + rank] = kv[:, :rank]
+        proj[:, spec.q_cols + R:spec.q_cols + R + rot_dim] = kv[:, rank:]
+        at = torch.arange(lens[0] - new, lens[0]) if new else torch.tensor(lens) - 1
+        r64 = lambda t: t.to(dtype).double()
+        want_q = plain.rotate(r64(q[..., dim:]), at, raw)
+        want_c = plain.rms_norm(r64(kv[:, :rank]), w.double(), 1e-3)
+        want_k = plain.rotate(r64(kv[:, rank:]), at, raw)
+        tol = dict(atol=2e-3 if at.max() > 1000 else 1e-4, rtol=1e-4) if dtype == F32 else dict(atol=3e-2, rtol=1e-2)
+        norm = torch.zeros(R)
+        norm[:rank] = w
+        indptr = torch.tensor([0, new], dtype=torch.int32, device=dev) if new else None
+        for in_place in (False, True):
+            pages = RowPages([torch.zeros(n, spec.row_cols) for n in lens], dtype, ps, dev, seed)
+            p, status = proj.to(dtype).to(dev), ops.new_status(dev)
+            q_out = None if in_place else torch.zeros(rows, heads, spec.row_cols, dtype=dtype, device=dev)
+            lo.latent_append(p, spec, pages.table, pages.pages, norm.to(dev), rotation.frequencies().to(dev), indptr, q_out,
+                             status=status)
+            ops.raise_on_status(status)
+            turned = p[:, :spec.q_cols].view(rows, heads, -1)[:, :, d:] if in_place else q_out[:, :, R:]
+            torch.testing.assert_close(turned[..., :rot_dim].double().cpu(), want_q, **tol)
+            for b in range(len(lens)):
+                row = pages.row(b)[-(new or 1):].double().cpu()
+                mine = slice(0, rows) if new else slice(b, b + 1)
+                torch.testing.assert_close(row[:, :rank], want_c[mine], **tol)
+                torch.testing.assert_close(row[:, R:R + rot_dim], want_k[mine], **tol)
+                assert (pages.row(b)[:-(new or 1)] == 0).all()
