@@ -177,3 +177,203 @@ def test_append_rotates_and_normalises(cuda_device, dtype):
                 torch.testing.assert_close(row[:, :rank], want_c[mine], **tol)
                 torch.testing.assert_close(row[:, R:R + rot_dim], want_k[mine], **tol)
                 assert (pages.row(b)[:-(new or 1)] == 0).all()
+
+
+# ---- the recurrence
+def _lru_case(spec, tokens, seed):
+    """Inputs of a sequence in true sizes, and the same padded block by block."""
+    from kinetics_b200.layer_ops import pad8
+    g = torch.Generator().manual_seed(seed)
+    B, n, bs = spec.blocks, spec.block, pad8(spec.block)
+    c = dict(x=torch.randn(tokens, B * n, generator=g), y=2 * torch.randn(tokens, B * n, generator=g),
+             w=torch.randn(B * n, spec.taps, generator=g), b=torch.randn(B * n, generator=g),
+             ra=torch.randn(B, n, n, generator=g) / n ** 0.5, ri=torch.randn(B, n, n, generator=g) / n ** 0.5,
+             rab=torch.randn(B, n, generator=g), rib=torch.randn(B, n, generator=g),
+             lam=3 * torch.randn(B * n, generator=g) - 3)
+
+    def spread(t, fill=0.0):                                  # [..., B * n] -> [..., B * bs]
+        out = torch.full((*t.shape[:-1], B, bs), fill)
+        out[..., :n] = t.view(*t.shape[:-1], B, n)
+        return out.flatten(-2)
+    return c, spread
+
+
+def _lru_plain(c, dtype):
+    r = lambda t: t.to(dtype).double()
+    x, y = r(c["x"]), r(c["y"])
+    u, _ = plain.causal_conv(x, x.new_zeros(c["w"].shape[1] - 1, x.shape[1]), c["w"].double(), c["b"].double())
+    u = r(u)
+    gate = lambda w, b: plain.block_gate(u, r(w), b.double())
+    s, _ = plain.linear_recurrence(gate(c["ra"], c["rab"]), gate(c["ri"], c["rib"]), u, c["lam"].double(), torch.zeros(x.shape[1]).double())
+    return s * plain.gelu_tanh(y)
+
+
+class _Lru:
+    """Drives conv, gate products and scan over one manager-like set of slots."""
+
+    def __init__(self, spec, cases, spread, dtype, dev, slots):
+        from kinetics_b200.layer_ops import pad8
+        c, n, bs = cases[0], spec.block, pad8(spec.block)
+        self.spec, self.dtype, self.dev = spec, dtype, dev
+        put = lambda t: t.float().to(dev).contiguous()
+        self.w, self.b = put(spread(c["w"].t())), put(spread(c["b"]))
+        gates = torch.zeros(spec.blocks, 2, bs, bs)
+        gates[:, 0, :n, :n], gates[:, 1, :n, :n] = c["ra"], c["ri"]
+        self.gates = gates.view(spec.blocks, 2 * bs, bs).to(dtype).to(dev)
+        self.rb, self.ib = put(spread(c["rab"].flatten())), put(spread(c["rib"].flatten()))
+        self.decay = put(spread(8 * torch.log1p(torch.exp(c["lam"].double()))))
+        self.state = torch.full((slots, spec.cols), float("nan"), device=dev)       # a new sequence reads none of it
+        self.ring = torch.full((slots, spec.taps, spec.cols), float("nan"), device=dev, dtype=dtype)
+
+    def run(self, y, x, table, slots, new=None):
+        from kinetics_b200 import layer_ops as lo, ops
+        proj = torch.cat((y, x), dim=1).to(self.dtype).to(self.dev)
+        status, slots = ops.new_status(self.dev), torch.tensor(slots, dtype=torch.int32, device=self.dev)
+        kw = dict(new_indptr=None if new is None else torch.tensor([0, new], dtype=torch.int32, device=self.dev),
+                  max_new=new or 1, status=status)
+        u = lo.lru_conv(proj, self.spec, table, slots, self.w, self.b, self.ring, **kw)
+        z = lo.lru_gate_products(u, self.gates, self.spec)
+        out = lo.lru_scan(z, u, proj, self.spec, table, slots, self.rb, self.ib, self.decay, self.state, **kw)
+        ops.raise_on_status(status)
+        return out.double().cpu()
+
+
+def _length_table(lens, dev, ps=16):
+    from kinetics_b200.layer_ops import PageTable
+    pages = [(n + ps - 1) // ps for n in lens]
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device=dev)
+    indptr = [sum(pages[:i]) for i in range(len(lens) + 1)]
+    return PageTable(i32(list(range(sum(pages)))), i32(indptr), i32([n - (c - 1) * ps for n, c in zip(lens, pages)]), ps, sum(pages))
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+@pytest.mark.parametrize("blocks,block,taps", [(3, 20, 4), (1, 48, 2), (2, 17, 1), (4, 8, 7), (2, 80, 4), (1, 16, 30)])
+def test_recurrence_in_portions(cuda_device, dtype, blocks, block, taps):
+    from kinetics_b200.layer_ops import LruSpec
+    spec = LruSpec(blocks, block, taps)
+    total = 300
+    c, spread = _lru_case(spec, total, blocks + taps)
+    want = spread(_lru_plain(c, dtype).float()).double()
+    y, x = spread(c["y"]), spread(c["x"])
+    lru = _Lru(spec, [c], spread, dtype, cuda_device, 3)
+    for slot, sizes in enumerate([[300], [2] * 150, [127, 1, 2, 129, 3, 16, 22]]):
+        got, at = [], 0
+        for n in sizes:
+            got.append(lru.run(y[at:at + n], x[at:at + n], _length_table([at + n], cuda_device), [slot], n if n > 1 else None))
+            at += n
+        err = (torch.cat(got) - want).pow(2).mean(-1).sqrt() / rms(want)
+        assert err.max() < (2e-5 if dtype == F32 else 2e-2), (sizes, float(err.max()))
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_recurrence_of_unequal_sequences(cuda_device, dtype):
+    # prompts of different lengths, then steps of all of them together in changing order; then a slot is used again
+    from kinetics_b200.layer_ops import LruSpec
+    spec, lens, steps = LruSpec(2, 24, 4), [1, 2, 5, 70], 40
+    cases = []
+    for i, n in enumerate(lens + [30]):
+        c, spread = _lru_case(spec, 1, 50)                    # the same weights, other inputs
+        g = torch.Generator().manual_seed(i)
+        c["x"], c["y"] = torch.randn(n + steps, spec.blocks * spec.block, generator=g), torch.randn(n + steps, spec.blocks * spec.block, generator=g)
+        cases.append(c)
+    lru = _Lru(spec, cases, spread, dtype, cuda_device, 6)
+    slot_of, got = [4, 0, 5, 2], [[] for _ in cases]
+
+    def prompt(i, n, slot):
+        c = cases[i]
+        got[i].append(lru.run(spread(c["y"][:n]), spread(c["x"][:n]), _length_table([n], cuda_device), [slot], n if n > 1 else None))
+    for i, n in enumerate(lens):
+        prompt(i, n, slot_of[i])
+    for t in range(steps):
+        order = [(k + t) % 4 for k in range(4)]
+        rows = lambda key: torch.cat([spread(cases[i][key][lens[i] + t:lens[i] + t + 1]) for i in order])
+        out = lru.run(rows("y"), rows("x"), _length_table([lens[i] + t + 1 for i in order], cuda_device), [slot_of[i] for i in order])
+        for k, i in enumerate(order):
+            got[i].append(out[k:k + 1])
+    prompt(4, 30, slot_of[3])
+    for i, n in enumerate(lens + [30]):
+        want = spread(_lru_plain(cases[i], dtype).float()).double()
+        mine = torch.cat(got[i])
+        err = (mine - want[:mine.shape[0]]).pow(2).mean(-1).sqrt() / rms(want)
+        assert err.max() < (2e-5 if dtype == F32 else 2e-2), (i, float(err.max()))
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_long_memory_and_short_memory(cuda_device, dtype):
+    # decays from "forgets at once" to "keeps for the whole sequence": the series and the difference in sqrt(1 - a^2)
+    from kinetics_b200.layer_ops import LruSpec
+    spec, total = LruSpec(1, 64, 4), 2000
+    c, spread = _lru_case(spec, total, 9)
+    c["lam"] = torch.linspace(-14, 4, 64)
+    want = _lru_plain(c, dtype)
+    got = _Lru(spec, [c], spread, dtype, cuda_device, 1).run(c["y"], c["x"], _length_table([total], cuda_device), [0], total)
+    err = (got - want).pow(2).mean(0).sqrt() / want.pow(2).mean(0).sqrt()
+    assert err.max() < (1e-4 if dtype == F32 else 3e-2), err
+
+
+# ---- feed-forward pieces
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_gated_rows_and_scale_cap(cuda_device, dtype):
+    from kinetics_b200 import layer_ops as lo
+    g = torch.Generator().manual_seed(0)
+    x = (4 * torch.randn(37, 2 * 88, generator=g)).to(dtype)
+    a, b = x[:, :88].double(), x[:, 88:].double()
+    tol = dict(rtol=1e-5, atol=1e-5) if dtype == F32 else dict(rtol=1e-2, atol=1e-3)
+    got = lo.gated_rows(x.to(cuda_device)).double().cpu()
+    torch.testing.assert_close(got, a * plain.sigmoid(a) * b, **tol)
+    got = lo.gated_rows(x.to(cuda_device), lo.GateSpec(1.5, 1.702, 1.0)).double().cpu()
+    a, b = a.clamp(max=1.5), b.clamp(-1.5, 1.5)
+    torch.testing.assert_close(got, a * plain.sigmoid(1.702 * a) * (b + 1), **tol)
+    z = 50 * torch.randn(5, 33, generator=g)
+    torch.testing.assert_close(lo.scale_cap(z.clone().to(cuda_device), 0.3, 9.0).cpu(), 9 * torch.tanh(z * 0.3 / 9), rtol=1e-5, atol=1e-5)
+    torch.testing.assert_close(lo.scale_cap(z.clone().to(cuda_device), 0.3, 0.0).cpu(), z * 0.3)
+
+
+@pytest.mark.parametrize("dtype", [F32, BF])
+def test_experts_with_clamped_gates_and_shares_of_the_whole_softmax(cuda_device, dtype):
+    from kinetics_b200 import layer_ops as lo
+    from kinetics_b200.layer_ops import GateSpec, MoeSpec
+    for rows, E, top, C, F, limit in [(5, 6, 2, 72, 40, 0.8), (300, 16, 3, 256, 64, 2.0), (700, 1, 1, 64, 32, 0.5), (64, 9, 9, 40, 24, 5.0)]:
+        g = torch.Generator().manual_seed(rows)
+        h = torch.randn(rows, C, generator=g).to(dtype)
+        # rows of one direction each: their experts stand far apart, so that rounding decides nothing
+        router = (torch.randn(E, C, generator=g) * (3.0 / C ** 0.5)).to(dtype)
+        gate, up, down = (torch.randn(E, *s, generator=g).div(s[1] ** 0.5).to(dtype) for s in ((F, C), (F, C), (C, F)))
+        spec = MoeSpec(E, top, C, F, score_all=True, gate=GateSpec(limit, 1.702, 1.0))
+        d = lambda t: t.to(cuda_device)
+        for variant in (0, 1):
+            r = lo.moe_route(d(h), d(router), None, spec, variant=variant)
+            y = lo.moe_experts(d(h), d(torch.stack((gate, up), dim=2).contiguous()), d(down), r, spec, variant=variant)
+            ids, weights = plain.route(h.double(), router.double(), top)
+            got_ids, got_w = r.ids.long().cpu(), r.weights.double().cpu()
+            same = (got_ids == ids).all(dim=1)
+            assert same.double().mean() > (0.999 if dtype == F32 else 0.97)
+            torch.testing.assert_close(got_w[same], weights[same], rtol=1e-4, atol=1e-5)
+            want = torch.zeros(rows, C).double()
+            for e in range(E):
+                at, place = (got_ids == e).nonzero(as_tuple=True)
+                if at.numel():
+                    part = plain.expert(h[at].double(), gate[e].double(), up[e].double(), down[e].double(), limit)
+                    want[at] += got_w[at, place].unsqueeze(1) * part
+            err = (y.double().cpu().sum(dim=1) - want).pow(2).mean(-1).sqrt() / rms(want)
+            assert err.max() < (1e-5 if dtype == F32 else 2e-2), float(err.max())
+
+
+def test_stream_without_norms_in_front(cuda_device):
+    from kinetics_b200 import layer_ops as lo, ops
+    g = torch.Generator().manual_seed(1)
+    rows, C, eps = 9, 72, 1e-3
+    table, tokens = torch.randn(50, C, generator=g), torch.randint(0, 50, (rows,), generator=g)
+    w, y = torch.randn(C, generator=g), torch.randn(rows, 3, C, generator=g)
+    dev = cuda_device
+    for dtype in (F32, BF):
+        x, h, status = torch.empty(rows, C, device=dev), torch.empty(rows, C, dtype=dtype, device=dev), ops.new_status(dev)
+        lo.residual_norm(x, h, C, eps, tokens=tokens.to(dev), embed=table.to(dtype).to(dev), embed_scale=2.5, center=False, status=status)
+        want = table.to(dtype)[tokens].double() * 2.5
+        torch.testing.assert_close(x.double().cpu(), want, rtol=1e-6, atol=1e-6)
+        assert torch.equal(h, x.to(dtype))
+        lo.residual_norm(x, h, C, eps, y=y.to(dtype).to(dev), parts=3, post=(w.to(dev), None), center=False, status=status)
+        want = want + plain.rms_norm(y.to(dtype).double().sum(1), w.double(), eps)
+        torch.testing.assert_close(x.double().cpu(), want, rtol=1e-5, atol=1e-5)
+        assert torch.equal(h, x.to(dtype))
+        ops.raise_on_status(status)
