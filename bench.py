@@ -108,12 +108,12 @@ def parse():
     ap.add_argument("--prefill-tokens", type=int, default=4096, help="--micro prefill: new tokens per prompt")
     ap.add_argument("--prefill-history", type=int, default=0,
                     help="--micro prefill: tokens every prompt already holds in its pages (a later chunk of a long prompt)")
-    ap.add_argument("--micro", default="", choices=["", "select", "exchange", "prefill", "gifetar"],
+    ap.add_argument("--micro", default="", choices=["", "select", "exchange", "prefill", "gifetar", "munadra"],
                     help="time one kernel alone on the workload's shapes (select: only the page summaries are "
                          "allocated, so the full batch fits in a few GB; exchange: the NVLink exchange kernels "
                          "on [batch, hidden] under torchrun, every form, beside NCCL; gifetar: prefill and decode of "
                          "Gifetar layers, kernel by kernel, beside DecoderStack at equal size)")
-    ap.add_argument("--only-kernel", default="", help="--micro gifetar: time only the kernels whose name holds this")
+    ap.add_argument("--only-kernel", default="", help="--micro gifetar, munadra: time only the kernels whose name holds this")
     return ap.parse_args()
 
 
@@ -1200,6 +1200,9 @@ def main():
         return run_micro_exchange(args)
     if args.micro == "prefill":
         return run_micro_prefill(args)
+    if args.micro == "munadra":
+        import bench_munadra
+        return emit(bench_munadra.run(args, ClockSampler))
     if args.micro == "gifetar":
         import bench_gifetar
         return emit(bench_gifetar.run(args, ClockSampler))
