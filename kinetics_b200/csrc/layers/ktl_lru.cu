@@ -2,17 +2,17 @@
 // sequence's next tokens or one token of every sequence.  State, gates and decays are fp32.
 //
 // The convolution keeps its newest `taps` inputs in a ring by position: a step writes the place of the input that has
-// just left the window, which nobody reads.  The prompt's scan is one pass: a CTA owns 16 channels and walks the tokens
-// in tiles; a thread runs 8 tokens of a channel, a warp shuffle joins the 16 runs of a tile, and the carry stays in a
-// register.  The next tile's loads are in flight meanwhile.
+// just left the window, which nobody reads.  The prompt's scan is one pass over its inputs: the CTAs of a cluster take
+// consecutive tiles of tokens and exchange the tiles' products and end states through distributed shared memory.
+#include "../ktk_umma.cuh"
 #include "ktl_common.cuh"
 
 namespace ktk {
 
 constexpr int kLcThreads = 64;
 constexpr int kLcChunk = 16;            // tokens per thread of the convolution
-constexpr int kLsChan = 16, kLsSegs = 16, kLsRun = 8;
-constexpr int kLsThreads = kLsChan * kLsSegs, kLsTile = kLsSegs * kLsRun;
+constexpr int kLsWarps = 8, kLsRun = 8;  // warps of a scan CTA, tokens of a warp
+constexpr int kLsThreads = kLsWarps * 32, kLsTile = kLsWarps * kLsRun, kLsMaxCluster = 8;
 constexpr int kLdThreads = 128;
 
 // what a sequence runs now: rows [row0, row0 + n), of positions base ..; false if the table or the slot is malformed
@@ -98,6 +98,19 @@ lru_conv_kernel(const T* __restrict__ x, int64_t row_stride, const int32_t* __re
 }
 
 // ---- gates and the recurrence ----
+// the float that CTA `cta` of the cluster keeps at the place of *p
+__device__ __forceinline__ float peer_f32(const float* p, uint32_t cta) {
+    uint32_t at;
+    float v;
+    asm volatile("mapa.shared::cluster.u32 %0, %1, %2;" : "=r"(at) : "r"(smem_u32(p)), "r"(cta));
+    asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(at) : "memory");
+    return v;
+}
+__device__ __forceinline__ float sqrt_approx(float x) {
+    float y;
+    asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
 template <bool FAST> __device__ __forceinline__ float exp_of(float x) { return FAST ? __expf(x) : expf(x); }
 template <bool FAST> __device__ __forceinline__ float sigmoid_of(float x) {
     return FAST ? __fdividef(1.0f, 1.0f + __expf(-x)) : 1.0f / (1.0f + expf(-x));
@@ -112,7 +125,7 @@ template <bool FAST>
 __device__ __forceinline__ void gates(float zr, float zi, float u, float rb, float ib, float decay, float& a, float& g) {
     const float x = sigmoid_of<FAST>(zr + rb) * decay;                    // -log a
     a = exp_of<FAST>(-x);
-    g = sqrtf(FAST ? one_minus_exp(2.0f * x, a * a) : -expm1f(-2.0f * x)) * sigmoid_of<FAST>(zi + ib) * u;
+    g = (FAST ? sqrt_approx(one_minus_exp(2.0f * x, a * a)) : sqrtf(-expm1f(-2.0f * x))) * sigmoid_of<FAST>(zi + ib) * u;
 }
 // 0.5 y (1 + tanh z) = y / (1 + exp(-2 z)),  z = sqrt(2 / pi) (y + 0.044715 y^3)
 template <bool FAST> __device__ __forceinline__ float gelu_tanh(float y) {
@@ -128,22 +141,27 @@ struct LruParams {
     int64_t row_stride;
     const int32_t *new_indptr, *slots;
     int64_t num_slots, rows;
+    int max_new;
     const float *rb, *ib, *decay;
     float* state;
     void* out;
     int32_t* status;
 };
 
-// 16 channels of one sequence: thread (channel, segment) holds 8 consecutive tokens of a tile of 128.
+// 32 channels of one sequence: lane = channel, a warp runs 8 consecutive tokens, a CTA 64, the CTAs of a cluster consecutive
+// tiles of 64.  Per round of the cluster: local products and end states, joined over the CTA's warps in shared memory and
+// over the cluster's CTAs through theirs; then every warp replays its tokens from the state in front of them.
 template <typename T>
-__global__ void __launch_bounds__(kLsThreads, 2) lru_scan_kernel(const LruParams p) {
+__global__ void __launch_bounds__(kLsThreads, 4) lru_scan_kernel(const LruParams p) {
     constexpr bool FAST = sizeof(T) == 2;
-    __shared__ float seg_a[kLsSegs][kLsChan + 1], seg_s[kLsSegs][kLsChan + 1], in_s[kLsSegs][kLsChan + 1];
+    // by parity of the round, so that a round needs no barrier behind its last reads
+    __shared__ float warp_a[2][kLsWarps][32], warp_s[2][kLsWarps][32], tile_a[2][32], tile_s[2][32], before[2][32];
     Run r;
-    if (!run_of(p.t, p.new_indptr, p.slots, p.num_slots, blockIdx.y, p.status, r)) return;
+    if (!run_of(p.t, p.new_indptr, p.slots, p.num_slots, blockIdx.z, p.status, r)) return;      // uniform for the cluster
+    const int ctas = gridDim.x, rank = blockIdx.x;
     const int bs = p.a.block_stride, width = p.a.blocks * bs;
-    const int tid = threadIdx.x, ch = tid % kLsChan, seg = tid / kLsChan;
-    const int c = blockIdx.x * kLsChan + ch;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int c = blockIdx.y * 32 + lane;
     const bool on = c < width;
     const int blk = on ? c / bs : 0, cc = on ? c - blk * bs : 0;
     const float* z = p.z + ((int64_t)blk * p.rows + r.row0) * (2 * bs) + cc;
@@ -151,64 +169,67 @@ __global__ void __launch_bounds__(kLsThreads, 2) lru_scan_kernel(const LruParams
     const T* y = (const T*)p.y + r.row0 * p.row_stride + (on ? c : 0);
     T* out = (T*)p.out + r.row0 * width + c;
     const float rb = on ? p.rb[c] : 0.0f, ib = on ? p.ib[c] : 0.0f, decay = on ? p.decay[c] : 0.0f;
-    // a thread of segment s, channel `ch` joins; lane = (channel of the pair, segment): a warp holds two channels
-    const int lane = tid & 31, jch = (tid >> 5) * 2 + (lane >> 4), jseg = lane & 15;
-    const int jc = blockIdx.x * kLsChan + jch;
-    float carry = jc < width && r.base > 0 ? p.state[(int64_t)r.slot * width + jc] : 0.0f;
-
-    float zr[kLsRun], zi[kLsRun];
-    T uu[kLsRun], yy[kLsRun];
-    auto fetch = [&](int tile) {
+    float carry = on && r.base > 0 ? p.state[(int64_t)r.slot * width + c] : 0.0f;      // behind the previous round
+    const int rounds = (r.n + ctas * kLsTile - 1) / (ctas * kLsTile);
+    for (int it = 0; it < rounds; ++it) {
+        const int par = it & 1, i0 = (it * ctas + rank) * kLsTile + warp * kLsRun;
+        float a[kLsRun], g[kLsRun], A = 1.0f, S = 0.0f;
+        {
+            float zr[kLsRun], zi[kLsRun];
+            T uu[kLsRun];
 #pragma unroll
-        for (int k = 0; k < kLsRun; ++k) {
-            const int i = tile * kLsTile + seg * kLsRun + k;
-            if (on && i < r.n) {
-                zr[k] = __ldcs(z + (int64_t)i * (2 * bs));
-                zi[k] = __ldcs(z + (int64_t)i * (2 * bs) + bs);
-                uu[k] = u[(int64_t)i * width];
-                yy[k] = y[(int64_t)i * p.row_stride];
+            for (int k = 0; k < kLsRun; ++k) {
+                const bool have = on && i0 + k < r.n;
+                const int64_t i = have ? i0 + k : 0;
+                zr[k] = have ? __ldcs(z + i * (2 * bs)) : 0.0f;
+                zi[k] = have ? __ldcs(z + i * (2 * bs) + bs) : 0.0f;
+                uu[k] = u[i * width];
             }
-        }
-    };
-    const int tiles = (r.n + kLsTile - 1) / kLsTile;
-    fetch(0);
-    for (int tile = 0; tile < tiles; ++tile) {
-        float a[kLsRun], g[kLsRun], yg[kLsRun], A = 1.0f, S = 0.0f;
-        const int i0 = tile * kLsTile + seg * kLsRun;
 #pragma unroll
-        for (int k = 0; k < kLsRun; ++k) {
-            a[k] = 1.0f;
-            g[k] = yg[k] = 0.0f;
-            if (on && i0 + k < r.n) {
+            for (int k = 0; k < kLsRun; ++k) {
                 gates<FAST>(zr[k], zi[k], to_f32(uu[k]), rb, ib, decay, a[k], g[k]);
-                yg[k] = gelu_tanh<FAST>(to_f32(yy[k]));
+                if (!(on && i0 + k < r.n)) { a[k] = 1.0f; g[k] = 0.0f; }
+                A *= a[k];
+                S = fmaf(a[k], S, g[k]);
             }
-            A *= a[k];
-            S = fmaf(a[k], S, g[k]);
         }
-        if (tile + 1 < tiles) fetch(tile + 1);
-        seg_a[seg][ch] = A;
-        seg_s[seg][ch] = S;
-        __syncthreads();
-        float ja = seg_a[jseg][jch], js = seg_s[jseg][jch];
+        warp_a[par][warp][lane] = A;
+        warp_s[par][warp][lane] = S;
+        T yy[kLsRun];                                      // in flight over the barriers
 #pragma unroll
-        for (int o = 1; o < kLsSegs; o <<= 1) {            // inclusive join over the 16 lanes of a channel
-            const float pa = __shfl_up_sync(0xffffffffu, ja, o, kLsSegs), ps = __shfl_up_sync(0xffffffffu, js, o, kLsSegs);
-            if (jseg >= o) { js = fmaf(ja, ps, js); ja *= pa; }
-        }
-        const float end = fmaf(ja, carry, js);             // state behind segment jseg
-        const float before = __shfl_up_sync(0xffffffffu, end, 1, kLsSegs);
-        in_s[jseg][jch] = jseg == 0 ? carry : before;
-        carry = __shfl_sync(0xffffffffu, end, kLsSegs - 1, kLsSegs);
+        for (int k = 0; k < kLsRun; ++k) yy[k] = y[(on && i0 + k < r.n ? (int64_t)(i0 + k) : 0) * p.row_stride];
         __syncthreads();
-        S = in_s[seg][ch];
+        if (warp == 0) {
+            A = 1.0f; S = 0.0f;
+#pragma unroll
+            for (int w = 0; w < kLsWarps; ++w) {
+                const float wa = warp_a[par][w][lane];
+                S = fmaf(wa, S, warp_s[par][w][lane]);
+                A *= wa;
+            }
+            tile_a[par][lane] = A;
+            tile_s[par][lane] = S;
+        }
+        cluster_sync();
+        if (warp == 0) {
+            float mine = carry;
+            for (int k = 0; k < ctas; ++k) {
+                if (k == rank) mine = carry;
+                carry = fmaf(peer_f32(&tile_a[par][lane], k), carry, peer_f32(&tile_s[par][lane], k));
+            }
+            before[par][lane] = mine;
+        }
+        __syncthreads();
+        S = before[par][lane];
+        for (int w = 0; w < warp; ++w) S = fmaf(warp_a[par][w][lane], S, warp_s[par][w][lane]);
 #pragma unroll
         for (int k = 0; k < kLsRun; ++k) {
             S = fmaf(a[k], S, g[k]);
-            if (on && i0 + k < r.n) out[(int64_t)(i0 + k) * width] = from_f32<T>(S * yg[k]);
+            if (on && i0 + k < r.n) out[(int64_t)(i0 + k) * width] = from_f32<T>(S * gelu_tanh<FAST>(to_f32(yy[k])));
         }
     }
-    if (jc < width && jseg == 0) p.state[(int64_t)r.slot * width + jc] = carry;
+    if (warp == 0 && rank == 0 && on) p.state[(int64_t)r.slot * width + c] = carry;
+    cluster_sync();                                        // no CTA leaves while another may read its totals
 }
 
 // One token of every sequence: a thread per channel.
@@ -234,7 +255,7 @@ static int check_lru(const ktk_lru* a, const ktk_paged* t, const int32_t* new_in
                      int64_t row_stride, int64_t col, int64_t num_slots, const char* who) {
     if (a == nullptr || t == nullptr || a->blocks <= 0 || a->block <= 0 || a->block_stride < a->block ||
         a->block_stride % 8 != 0 || a->taps <= 0 || a->taps > 1024 || (a->dtype != KTK_F32 && a->dtype != KTK_BF16) ||
-        (int64_t)a->blocks * a->block_stride > (1 << 24) || t->page_size <= 0 || t->batch < 0 || t->batch > 65535) {
+        (int64_t)a->blocks * a->block_stride > (1 << 20) || t->page_size <= 0 || t->batch < 0 || t->batch > 65535) {
         set_error("%s: bad sizes", who);
         return KTK_ERR_ARG;
     }
@@ -265,8 +286,23 @@ static int conv_launch(const void* x, int64_t row_stride, const int32_t* ni, int
 
 template <typename T> static int scan_launch(const LruParams& p, cudaStream_t st) {
     const int width = p.a.blocks * p.a.block_stride;
-    if (p.new_indptr)
-        lru_scan_kernel<T><<<dim3((unsigned)((width + kLsChan - 1) / kLsChan), (unsigned)p.t.batch), kLsThreads, 0, st>>>(p);
+    if (p.new_indptr) {
+        // as many CTAs along the sequence as stay resident together and have tokens
+        const int64_t groups = (width + 31) / 32, tiles = (p.max_new + kLsTile - 1) / kLsTile;
+        int ctas = kLsMaxCluster;
+        while (ctas > 1 && (ctas > tiles || groups * p.t.batch * ctas > (int64_t)sm_count() * 4)) ctas /= 2;
+        cudaLaunchConfig_t cfg{};
+        cfg.gridDim = dim3((unsigned)ctas, (unsigned)groups, (unsigned)p.t.batch);
+        cfg.blockDim = dim3(kLsThreads);
+        cfg.stream = st;
+        cudaLaunchAttribute attr{};
+        attr.id = cudaLaunchAttributeClusterDimension;
+        attr.val.clusterDim.x = ctas;
+        attr.val.clusterDim.y = attr.val.clusterDim.z = 1;
+        cfg.attrs = &attr;
+        cfg.numAttrs = 1;
+        KTK_CUDA_TRY(cudaLaunchKernelEx(&cfg, lru_scan_kernel<T>, p), "ktk_lru_scan");
+    }
     else
         lru_step_kernel<T><<<dim3((unsigned)((width + kLdThreads - 1) / kLdThreads), (unsigned)p.t.batch), kLdThreads, 0, st>>>(p);
     KTK_CUDA_TRY(cudaGetLastError(), "ktk_lru_scan");
@@ -312,6 +348,6 @@ extern "C" int ktk_lru_scan(const float* z, const void* u, const void* proj, int
     }
     const size_t size = shape->dtype == KTK_F32 ? 4 : 2;
     const LruParams p{*shape, *table, z, u, (const char*)proj + y_col * size, row_stride, new_indptr, slots, num_slots, rows,
-                      rb, ib, decay, state, out, status};
+                      max_new, rb, ib, decay, state, out, status};
     return shape->dtype == KTK_F32 ? scan_launch<float>(p, (cudaStream_t)stream) : scan_launch<__nv_bfloat16>(p, (cudaStream_t)stream);
 }
