@@ -135,6 +135,31 @@ __device__ __forceinline__ void tmem_st16(uint32_t taddr, const float (&v)[16]) 
         : "memory");
 }
 
+// 16 lanes of tensor memory from taddr's on, 8 X columns, by a whole warp: thread i gets columns 8 k + 2 (i % 4) and the next
+// of lane i / 4 in r[4 k], r[4 k + 1], of lane i / 4 + 8 in r[4 k + 2], r[4 k + 3]
+template <int X> struct RowPairs;
+template <> struct RowPairs<2> {
+    static __device__ __forceinline__ void load(uint32_t taddr, uint32_t (&r)[8]) {
+        asm volatile("tcgen05.ld.sync.aligned.16x256b.x2.b32 {%0, %1, %2, %3, %4, %5, %6, %7}, [%8];\n\t"
+                     "tcgen05.wait::ld.sync.aligned;"
+                     : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]) : "r"(taddr));
+    }
+};
+template <> struct RowPairs<4> {
+    static __device__ __forceinline__ void load(uint32_t taddr, uint32_t (&r)[16]) {
+        asm volatile("tcgen05.ld.sync.aligned.16x256b.x4.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15}, [%16];\n\t"
+                     "tcgen05.wait::ld.sync.aligned;"
+                     : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]) : "r"(taddr));
+    }
+};
+template <> struct RowPairs<8> {
+    static __device__ __forceinline__ void load(uint32_t taddr, uint32_t (&r)[32]) {
+        asm volatile("tcgen05.ld.sync.aligned.16x256b.x8.b32 {%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, %16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];\n\t"
+                     "tcgen05.wait::ld.sync.aligned;"
+                     : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]), "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]), "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]), "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31]) : "r"(taddr));
+    }
+};
+
 // One lane of a converged warp.  The issuing warps run their loops with all lanes and pick the lane only around the
 // instructions themselves: descriptors and barrier addresses can then stay in uniform registers, which is what the
 // tcgen05 instructions take; from a branch on the lane number every operand has to be moved there first.
@@ -162,6 +187,10 @@ __device__ __forceinline__ bool mbar_wait_fast(uint64_t* bar, uint32_t parity, v
     return false;
 }
 
+// The same for a converged warp: its lanes agree on the outcome and go on together.
+__device__ __forceinline__ bool mbar_wait_all(uint64_t* bar, uint32_t parity, volatile int* abort) {
+    return __all_sync(0xffffffffu, mbar_wait_fast(bar, parity, abort)) != 0;
+}
 // whether the phase has completed, without waiting
 __device__ __forceinline__ bool mbar_test(uint64_t* bar, uint32_t parity) {
     uint32_t ok;

@@ -9,8 +9,8 @@
 //                               two blocks in flight
 //     issuing warp              S_m[128 x 64] = Q_m . K^T, then O_m[128 x vdim] += P_m . V with P_m from tensor memory;
 //                               S of block j + 1 is issued before O += P . V of block j
-//     softmax thread            S row -> registers; scale, mask, 2^x against a reference that starts at the sink and
-//                               moves in jumps of at least 2^8; P as bf16 pairs over that S
+//     softmax thread            S row -> registers; scale, mask, 2^x against a reference, at first the largest of the sink
+//                               and the first block's scores, that moves in jumps of at least 2^8; P as bf16 pairs over that S
 // Tensor memory: S of two blocks and two tiles in columns [0, 256), O_1 and O_2 behind.  Every wait is bounded.
 #include "ktl_score.cuh"
 
@@ -74,7 +74,7 @@ attn_expanded_kernel(const ExpandedParams p, const __grid_constant__ CUtensorMap
 
     if (tid == 0) {
         for (int i = 0; i < 2; ++i) {
-            for (int m = 0; m < 2; ++m) { mbar_init(&bar_s[m][i], 1); mbar_init(&bar_p[m][i], kUmRows); }
+            for (int m = 0; m < 2; ++m) { mbar_init(&bar_s[m][i], 1); mbar_init(&bar_p[m][i], 4); }
             mbar_init(&bar_k[i], 1); mbar_init(&bar_v[i], 1);
             mbar_init(&bar_kfree[i], 1); mbar_init(&bar_vfree[i], 1);
             mbar_init(&bar_o[i], 1);
@@ -107,7 +107,7 @@ attn_expanded_kernel(const ExpandedParams p, const __grid_constant__ CUtensorMap
         const uint64_t q_desc = umma_desc(smem_u32(sQ), 0, 1024), k_desc = umma_desc(smem_u32(sK), 0, 1024);
         const uint64_t v_desc = umma_desc(smem_u32(sV), kAeKTile, 1024);
         auto wait = [&](uint64_t* bar, int round) {
-            return __all_sync(0xffffffffu, mbar_wait_fast(bar, round & 1, &abort_flag)) != 0;
+            return mbar_wait_all(bar, round & 1, &abort_flag);
         };
         auto issue_s = [&](int blk) {
             const int buf = blk & 1;
@@ -210,7 +210,7 @@ attn_expanded_kernel(const ExpandedParams p, const __grid_constant__ CUtensorMap
         for (int j = 0; j < mine; ++j) {
             const int buf = j & 1;
             const uint32_t s_col = tile * 128 + buf * kAeKeys;
-            if (!__all_sync(0xffffffffu, mbar_wait_fast(&bar_s[tile][buf], (j >> 1) & 1, &abort_flag))) { alive = false; break; }
+            if (!mbar_wait_all(&bar_s[tile][buf], (j >> 1) & 1, &abort_flag)) { alive = false; break; }
             tc_fence_after();
             float lo[32], hi[32];
             tmem_ld64(my + s_col, lo, hi);
@@ -227,7 +227,7 @@ attn_expanded_kernel(const ExpandedParams p, const __grid_constant__ CUtensorMap
             for (int c = 1; c < 32; ++c) mx = fmaxf(mx, fmaxf(lo[c], hi[c]));
             mx *= f;                                                   // f > 0
             float alpha = 1.0f;
-            if (mx > m_ref + kAeSlack) {
+            if (mx > m_ref + (j == 0 ? 0.0f : kAeSlack)) {
                 alpha = ex2(m_ref - mx);
                 m_ref = mx;
                 l_run *= alpha;
@@ -245,8 +245,7 @@ attn_expanded_kernel(const ExpandedParams p, const __grid_constant__ CUtensorMap
             }
             l_run += sum0 + sum1;
             if (j > 0 && __any_sync(0xffffffffu, alpha != 1.0f)) {
-                if (!mbar_wait_fast(&bar_vfree[(j - 1) & 1], ((j - 1) >> 1) & 1, &abort_flag)) alive = false;
-                __syncwarp();
+                if (!mbar_wait_all(&bar_vfree[(j - 1) & 1], ((j - 1) >> 1) & 1, &abort_flag)) alive = false;
                 tc_fence_after();
 #pragma unroll
                 for (int c = 0; c < VC * 64; c += 32) {
@@ -260,10 +259,10 @@ attn_expanded_kernel(const ExpandedParams p, const __grid_constant__ CUtensorMap
             tmem_st32_u32(my + s_col, packed);
             tmem_st_wait();
             tc_fence_before();
-            mbar_arrive(&bar_p[tile][buf]);
+            __syncwarp();
+            if (lane == 0) mbar_arrive(&bar_p[tile][buf]);
         }
-        if (mine > 0 && alive && !mbar_wait_fast(&bar_o[tile], 0, &abort_flag)) alive = false;
-        __syncwarp();
+        if (mine > 0 && alive && !mbar_wait_all(&bar_o[tile], 0, &abort_flag)) alive = false;
         tc_fence_after();
         if (mine > 0 && __all_sync(0xffffffffu, alive)) {
             float g = l_run > 0.0f ? 1.0f / l_run : 0.0f;

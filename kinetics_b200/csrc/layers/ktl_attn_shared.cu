@@ -8,9 +8,9 @@
 // One CTA per (split of the tokens, chunk of heads, group of rows).  Roles:
 //     loading warp     TMA: tiles of 64 tokens into a ring
 //     issuing warp     both products, in whatever order their inputs become ready
-//     softmax warps    thread = token: lanes 0..15 of warp w hold tokens 16 w ..; exponentials against a reference per
-//                      column that starts at the column's sink and moves only when a score exceeds it by 2^8
-// The sum of a column's weights stays spread over the tokens' threads until the end.  Tensor memory: S of two tiles, then
+//     softmax warps    warp w holds tokens 16 w .., two per thread; exponentials against a reference per column, at first the largest of its sink and the first tile's scores, that moves
+//                      only when a score exceeds it by 2^8
+// The sum of a column's weights stays spread over the threads until the end.  Tensor memory: S of two tiles, then
 // O^T in blocks of 128 columns of V.  Every wait is bounded.
 #include "ktl_score.cuh"
 
@@ -19,10 +19,10 @@ namespace ktk {
 constexpr int kAsTok = 64;
 constexpr int kAsThreads = 192;               // 4 softmax warps, the issuing warp, the loading warp
 constexpr int kAsChunk = kAsTok * 128;        // [64 tokens][64 columns]
-constexpr int kAsMaxStages = 8;
+constexpr int kAsMaxStages = 8, kAsMaxBars = 40;
 constexpr int kAsSmem = 232448 - 2048;        // for Q, the ring and P; static arrays and alignment aside
 constexpr int kAsMinTiles = 4;                // a split is not worth less
-constexpr int kAsMaxSplits = 256;
+constexpr int kAsMaxSplits = 256, kAsStartTiles = 2;
 constexpr int kAsMaxDim = 576, kAsMaxVdim = 512;
 constexpr float kAsSlack = 8.0f;
 constexpr float kAsNone = -1e30f;             // reference of a column without a sink
@@ -69,14 +69,15 @@ __global__ void __launch_bounds__(kAsThreads, 1)
 attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map, const int kc, const int stages,
                    const uint32_t tmem_cols) {
     extern __shared__ uint8_t as_raw[];
-    __shared__ __align__(8) uint64_t full[kAsMaxStages], free_[kAsMaxStages], bar_s[2], bar_p, bar_o;
+    // a stage has landed; a pair of its chunks has been read out
+    __shared__ __align__(8) uint64_t full[kAsMaxStages], free_[kAsMaxBars], bar_s[2], bar_p, bar_o;
     __shared__ __align__(16) float ref_s[N], alpha_s[N];
-    __shared__ int vis_s[N];
+    __shared__ __align__(16) int vis_s[N];
     __shared__ uint32_t tmem_base_s;
     __shared__ int abort_flag;
     uint8_t* sQ = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(as_raw) + 1023) & ~uintptr_t(1023));
     uint8_t* sK = sQ + kc * (N * 128);                  // [stage][chunk]
-    const int stage_bytes = kc * kAsChunk;
+    const int stage_bytes = kc * kAsChunk, pairs = (kc + 1) / 2;
     uint8_t* sP = sK + stages * stage_bytes;            // [64 tokens][N], rows of 128 bytes
     float* scratch = reinterpret_cast<float*>(sP);
 
@@ -103,7 +104,8 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
     const int ps = p.t.page_size;
 
     if (tid == 0) {
-        for (int i = 0; i < stages; ++i) { mbar_init(&full[i], 1); mbar_init(&free_[i], 1); }
+        for (int i = 0; i < stages; ++i) mbar_init(&full[i], 1);
+        for (int i = 0; i < stages * pairs; ++i) mbar_init(&free_[i], 1);
         mbar_init(&bar_s[0], 1); mbar_init(&bar_s[1], 1);
         mbar_init(&bar_p, 128);
         mbar_init(&bar_o, 1);
@@ -135,67 +137,70 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
     tc_fence_after();
     const uint32_t tmem = tmem_base_s, tmem_o = tmem + 2 * N;
     const int vblocks = (a.vdim_stride + kUmRows - 1) / kUmRows;
-    float l[N];
-#pragma unroll
-    for (int c = 0; c < N; ++c) l[c] = 0.0f;
 
     if (issuer) {
-        const int ksteps = (a.dim_stride + 15) / 16;
         const uint32_t idesc_s = umma_idesc_of(kAsTok, N, false, false), idesc_o = umma_idesc_of(kUmRows, N, true, true);
         const uint64_t q_desc = umma_desc(smem_u32(sQ), 0, 1024), k_desc = umma_desc(smem_u32(sK), 0, 1024);
         const uint64_t v_desc = umma_desc(smem_u32(sK), kAsChunk, 1024), p_desc = umma_desc(smem_u32(sP), 0, 1024);
         int s_at = 0, o_at = 0;                          // next tile of each product
-        uint32_t idle = 0;
+        int s_st = 0, o_st = 0;                          // their stages
+        uint32_t s_par = 0, idle = 0;
         while (o_at < n) {
-            bool did = false;
-            if (s_at < n && s_at <= o_at + 1 &&
-                __all_sync(0xffffffffu, mbar_test(&full[s_at % stages], (s_at / stages) & 1))) {
+            uint32_t ready = 0;
+            if (o_at < s_at && __all_sync(0xffffffffu, mbar_test(&bar_p, o_at & 1))) ready |= 1u;
+            if (s_at < n && s_at <= o_at + ((ready & 1u) ? 2 : 1) && __all_sync(0xffffffffu, mbar_test(&full[s_st], s_par))) ready |= 2u;
+            if (ready & 1u) {
                 tc_fence_after();
                 if (elect_one()) {
-                    const uint64_t ka = umma_desc_at(k_desc, (s_at % stages) * stage_bytes);
-                    for (int k = 0; k < ksteps; ++k)
-                        umma_f16(tmem + (s_at & 1) * N, umma_desc_at(ka, (k >> 2) * kAsChunk + (k & 3) * 32),
-                                 umma_desc_at(q_desc, (k >> 2) * (N * 128) + (k & 3) * 32), idesc_s, k > 0 ? 1u : 0u);
-                    umma_commit(&bar_s[s_at & 1]);
-                }
-                __syncwarp();
-                ++s_at;
-                did = true;
-            }
-            if (o_at < s_at && __all_sync(0xffffffffu, mbar_test(&bar_p, o_at & 1))) {
-                tc_fence_after();
-                if (elect_one()) {
-                    const uint64_t va = umma_desc_at(v_desc, (o_at % stages) * stage_bytes);
-                    for (int v = 0; v < vblocks; ++v)
+                    uint64_t va = umma_desc_at(v_desc, o_st * stage_bytes);
+                    uint32_t d = tmem_o;
+                    for (int v = 0; v < vblocks; ++v, d += N, va = umma_desc_at(va, 2 * kAsChunk)) {
 #pragma unroll
                         for (int k = 0; k < kAsTok / 16; ++k)
-                            umma_f16(tmem_o + v * N, umma_desc_at(va, 2 * v * kAsChunk + k * (16 * 128)),
-                                     umma_desc_at(p_desc, k * (16 * 128)), idesc_o, (o_at > 0 || k > 0) ? 1u : 0u);
-                    umma_commit(&free_[o_at % stages]);
+                            umma_f16(d, umma_desc_at(va, k * (16 * 128)), umma_desc_at(p_desc, k * (16 * 128)), idesc_o,
+                                     (o_at > 0 || k > 0) ? 1u : 0u);
+                        umma_commit(&free_[o_st * pairs + v]);
+                    }
                     umma_commit(&bar_o);
                 }
                 __syncwarp();
                 ++o_at;
-                did = true;
+                if (++o_st == stages) o_st = 0;
             }
-            if (did) { idle = 0; continue; }
-            if (++idle > (1u << 24) || ((idle & 63u) == 63u && *(volatile int*)&abort_flag)) {   // bounded, like every wait
+            if (ready & 2u) {
+                if (elect_one()) {
+                    uint64_t ka = umma_desc_at(k_desc, s_st * stage_bytes), qa = q_desc;
+                    const uint32_t d = tmem + (s_at & 1) * N;
+                    for (int c = 0; c < kc; ++c) {       // columns past `dim` are zero in Q and in K
+#pragma unroll
+                        for (int k = 0; k < 4; ++k)
+                            umma_f16(d, umma_desc_at(ka, k * 32), umma_desc_at(qa, k * 32), idesc_s, (c > 0 || k > 0) ? 1u : 0u);
+                        ka = umma_desc_at(ka, kAsChunk);
+                        qa = umma_desc_at(qa, N * 128);
+                    }
+                    umma_commit(&bar_s[s_at & 1]);
+                    for (int v = vblocks; v < pairs; ++v) umma_commit(&free_[s_st * pairs + v]);       // no values in these
+                }
+                __syncwarp();
+                ++s_at;
+                if (++s_st == stages) { s_st = 0; s_par ^= 1u; }
+            }
+            if (ready) { idle = 0; continue; }
+            if (++idle > (1u << 22) || ((idle & 63u) == 63u && *(volatile int*)&abort_flag)) {   // bounded, like every wait
                 abort_flag = 1;
                 break;
             }
         }
     } else if (loader) {
-        int issued = 0;
-        bool alive = true;
         if (lane == 0) {
             const int box = ps < kAsTok ? ps : kAsTok, pages = kAsTok / box;
+            int st = 0, issued = 0;
+            uint32_t par = 1;
+            bool alive = true;
             prefetch_tensormap(&k_map);
             for (int i = 0; i < n && alive; ++i) {
-                const int st = i % stages;
-                if (i >= stages && !mbar_wait_fast(&free_[st], (i / stages - 1) & 1, &abort_flag)) { alive = false; break; }
                 const int tok0 = (j0 + i) * kAsTok;
-                int z[kAsTok / 16];
-                uint32_t bytes = 0;
+                int z[kAsTok / 16], have = 0;
 #pragma unroll
                 for (int k = 0; k < kAsTok / 16; ++k) {
                     z[k] = -1;
@@ -203,18 +208,29 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
                     if (k < pages && tok < s.total) {
                         const int pg = p.t.kv_indices[s.start + tok / ps];
                         if (pg < 0 || pg >= p.t.num_pages) report(p.status, KTK_STATUS_BAD_PAGE);
-                        else { z[k] = pg; bytes += (uint32_t)(kc * box * 128); }
+                        else { z[k] = pg; ++have; }
                     }
                 }
-                if (bytes) mbar_arrive_expect_tx(&full[st], bytes);
-                else mbar_arrive(&full[st]);
-                uint8_t* dst = sK + st * stage_bytes;
+                const uint32_t bytes = (uint32_t)(have * box * 128 * kc);
+                uint64_t* bar = &full[st];
+                for (int c = 0; c < kc && alive; ++c) {
+                    if (i >= stages && (c & 1) == 0) alive = mbar_wait_fast(&free_[st * pairs + (c >> 1)], par, &abort_flag);
+                    if (!alive) break;
+                    if (c == 0) {
+                        if (bytes) mbar_arrive_expect_tx(bar, bytes);
+                        else mbar_arrive(bar);
+                    }
+                    uint8_t* dst = sK + st * stage_bytes + c * kAsChunk;
+                    if (pages == 1) {
+                        if (z[0] >= 0) tma_load_3d(dst, &k_map, bar, c * 64, 0, z[0]);
+                    } else {
 #pragma unroll
-                for (int k = 0; k < kAsTok / 16; ++k)
-                    if (z[k] >= 0)
-                        for (int c = 0; c < kc; ++c)
-                            tma_load_3d(dst + c * kAsChunk + k * box * 128, &k_map, &full[st], c * 64, 0, z[k]);
-                ++issued;
+                        for (int k = 0; k < kAsTok / 16; ++k)
+                            if (z[k] >= 0) tma_load_3d(dst + k * box * 128, &k_map, bar, c * 64, 0, z[k]);
+                    }
+                }
+                if (alive) ++issued;
+                if (++st == stages) { st = 0; par ^= 1u; }
             }
             if (abort_flag || !alive) {                  // the copies in flight still write shared memory
                 volatile int never = 0;
@@ -224,54 +240,62 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
         }
     } else {
         const uint32_t my = tmem + ((uint32_t)(warp * 32) << 16);
-        const bool on = lane < 16;
-        const int tok = warp * 16 + (lane & 15);         // within the tile
+        // a thread holds two tokens of the tile and, of every 8 columns, the two from 2 (lane % 4) on
+        const int tok = warp * 16 + (lane >> 2), col = 2 * (lane & 3);
         const float f = a.scale * kLog2eF;
         const int clean_end = base + first + 1;          // tokens before this are seen by every row of the CTA
+        float l[N / 4];
+#pragma unroll
+        for (int c = 0; c < N / 4; ++c) l[c] = 0.0f;
+        // waits that ran out raise abort_flag; the loop still runs to its end, so that no warp misses a barrier
         for (int j = 0; j < n; ++j) {
             const int at = (j0 + j) * kAsTok + tok;
-            // a wait that ran out raises abort_flag; the loop still runs to its end, so that no warp misses a barrier
-            mbar_wait_fast(&bar_s[j & 1], (j >> 1) & 1, &abort_flag);
-            __syncwarp();
+            mbar_wait_all(&bar_s[j & 1], (j >> 1) & 1, &abort_flag);
             tc_fence_after();
-            float t[N];
-            tmem_ld_cols<N>(my + (j & 1) * N, t);
+            uint32_t raw[N / 2];
+            RowPairs<N / 8>::load(my + (j & 1) * N, raw);
+            float t[N / 2];
             bool over = false;
             const bool clean = (j0 + j + 1) * kAsTok <= clean_end;
 #pragma unroll
-            for (int c = 0; c < N; c += 4) {
-                const float4 r4 = *reinterpret_cast<const float4*>(ref_s + c);
-                const float r[4] = {r4.x, r4.y, r4.z, r4.w};
-#pragma unroll
-                for (int e = 0; e < 4; ++e) {
-                    t[c + e] = on && (clean || at < vis_s[c + e]) ? t[c + e] * f : -INFINITY;
-                    over |= t[c + e] > r[e] + kAsSlack;
-                }
+            for (int k = 0; k < N / 8; ++k) {
+                const float2 r = *reinterpret_cast<const float2*>(ref_s + 8 * k + col);
+                const int2 v = clean ? make_int2(0x7fffffff, 0x7fffffff) : *reinterpret_cast<const int2*>(vis_s + 8 * k + col);
+                t[4 * k] = at < v.x ? __uint_as_float(raw[4 * k]) * f : -INFINITY;
+                t[4 * k + 1] = at < v.y ? __uint_as_float(raw[4 * k + 1]) * f : -INFINITY;
+                t[4 * k + 2] = at + 8 < v.x ? __uint_as_float(raw[4 * k + 2]) * f : -INFINITY;
+                t[4 * k + 3] = at + 8 < v.y ? __uint_as_float(raw[4 * k + 3]) * f : -INFINITY;
+                over |= fmaxf(t[4 * k], t[4 * k + 2]) > r.x + kAsSlack || fmaxf(t[4 * k + 1], t[4 * k + 3]) > r.y + kAsSlack;
             }
-            const bool move = any_of_softmax_warps(over);
-            if (j > 0) mbar_wait_fast(&bar_o, (j - 1) & 1, &abort_flag);      // P and O of the previous tile are settled
-            __syncwarp();
+            const bool move = any_of_softmax_warps(over || j == 0);
+            if (j > 0) mbar_wait_all(&bar_o, (j - 1) & 1, &abort_flag);       // P and O of the previous tile are settled
             if (move) {
                 // some reference moves: every column's largest score of the tile, then O and the sums are rescaled
 #pragma unroll
-                for (int c = 0; c < N; ++c) {
-                    float mx = t[c];
+                for (int k = 0; k < N / 8; ++k)
 #pragma unroll
-                    for (int o = 8; o > 0; o >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-                    if (lane == 0) scratch[warp * N + c] = mx;
-                }
+                    for (int e = 0; e < 2; ++e) {
+                        float mx = fmaxf(t[4 * k + e], t[4 * k + 2 + e]);
+#pragma unroll
+                        for (int o = 4; o <= 16; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+                        if (lane < 4) scratch[warp * N + 8 * k + col + e] = mx;
+                    }
                 softmax_warps_sync();
                 for (int c = tid; c < N; c += 128) {
                     const float old = ref_s[c];
                     const float mx = fmaxf(fmaxf(scratch[c], scratch[N + c]), fmaxf(scratch[2 * N + c], scratch[3 * N + c]));
-                    const float now = mx > old + kAsSlack ? mx : old;
+                    const float now = fmaxf(mx, old);
                     ref_s[c] = now;
                     alpha_s[c] = ex2(old - now);
                 }
                 softmax_warps_sync();
                 tc_fence_after();
 #pragma unroll
-                for (int c = 0; c < N; ++c) l[c] *= alpha_s[c];
+                for (int k = 0; k < N / 8; ++k) {
+                    const float2 al = *reinterpret_cast<const float2*>(alpha_s + 8 * k + col);
+                    l[2 * k] *= al.x;
+                    l[2 * k + 1] *= al.y;
+                }
                 if (j > 0)
                     for (int v = 0; v < vblocks; ++v) {
                         float o[N];
@@ -283,33 +307,38 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
                 tmem_st_wait();
             }
 #pragma unroll
-            for (int c = 0; c < N; c += 8) {
-                float e[8];
-#pragma unroll
-                for (int x = 0; x < 8; ++x) { e[x] = ex2(t[c + x] - ref_s[c + x]); l[c + x] += e[x]; }
-                if (on) Vec8<__nv_bfloat16>::store(reinterpret_cast<__nv_bfloat16*>(sP + swz(tok, c >> 3)), e);
+            for (int k = 0; k < N / 8; ++k) {
+                const float2 r = *reinterpret_cast<const float2*>(ref_s + 8 * k + col);
+                const float p0 = ex2(t[4 * k] - r.x), p1 = ex2(t[4 * k + 1] - r.y);
+                const float p2 = ex2(t[4 * k + 2] - r.x), p3 = ex2(t[4 * k + 3] - r.y);
+                l[2 * k] += p0 + p2;
+                l[2 * k + 1] += p1 + p3;
+                *reinterpret_cast<uint32_t*>(sP + swz(tok, k) + 2 * col) = pack_bf16(p0, p1);
+                *reinterpret_cast<uint32_t*>(sP + swz(tok + 8, k) + 2 * col) = pack_bf16(p2, p3);
             }
             const int left = s.total - (j0 + j) * kAsTok;
-            if (left < kAsTok && on && tok >= left) {    // rows behind the sequence may hold anything: 0 * x has to stay 0
+            if (left < kAsTok && lane < 16 && warp * 16 + lane >= left) {
+                // rows behind the sequence may hold anything: 0 * x has to stay 0
                 uint8_t* st = sK + (j % stages) * stage_bytes;
                 for (int c = 0; c < kc * 8; ++c)
-                    *reinterpret_cast<uint4*>(st + (c >> 3) * kAsChunk + swz(tok, c & 7)) = make_uint4(0u, 0u, 0u, 0u);
+                    *reinterpret_cast<uint4*>(st + (c >> 3) * kAsChunk + swz(warp * 16 + lane, c & 7)) = make_uint4(0u, 0u, 0u, 0u);
             }
             fence_proxy_async();
             tc_fence_before();
             mbar_arrive(&bar_p);
         }
-        if (n > 0) mbar_wait_fast(&bar_o, (n - 1) & 1, &abort_flag);
-        __syncwarp();
+        if (n > 0) mbar_wait_all(&bar_o, (n - 1) & 1, &abort_flag);
         tc_fence_after();
         // ---- sums over the tokens, then O^T: lane = column of V, register = (row, head)
 #pragma unroll
-        for (int c = 0; c < N; ++c) {
-            float v = l[c];
+        for (int k = 0; k < N / 8; ++k)
 #pragma unroll
-            for (int o = 8; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-            if (lane == 0) scratch[warp * N + c] = v;
-        }
+            for (int e = 0; e < 2; ++e) {
+                float v = l[2 * k + e];
+#pragma unroll
+                for (int o = 4; o <= 16; o <<= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+                if (lane < 4) scratch[warp * N + 8 * k + col + e] = v;
+            }
         softmax_warps_sync();
         for (int c = tid; c < N; c += 128) {
             float L = scratch[c] + scratch[N + c] + scratch[2 * N + c] + scratch[3 * N + c];
@@ -368,12 +397,23 @@ __global__ void __launch_bounds__(128) attn_shared_combine_kernel(const AttnPara
     const int64_t stride = as_partial_floats(a.vdim_stride);
     const float* w = p.ws + (row * a.heads + head) * p.splits * stride;
     const float sk = p.sink ? p.sink[head] * kLog2eF : kAsNone;
+    // every warp reads all the splits' references and sums, a lane some of them
+    const int lane = threadIdx.x & 31;
     float M = sk, L = 0.0f;
-    for (int s = 0; s < p.splits; ++s)
-        if (w[s * stride + 1] > 0.0f) M = fmaxf(M, w[s * stride]);
-    for (int s = threadIdx.x; s < p.splits; s += 128) weight[s] = w[s * stride + 1] > 0.0f ? ex2(w[s * stride] - M) : 0.0f;
+    for (int s = lane; s < p.splits; s += 32) {
+        const float2 ml = *reinterpret_cast<const float2*>(w + s * stride);
+        if (ml.y > 0.0f) M = fmaxf(M, ml.x);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) M = fmaxf(M, __shfl_xor_sync(0xffffffffu, M, o));
+    for (int s = lane; s < p.splits; s += 32) {
+        const float2 ml = *reinterpret_cast<const float2*>(w + s * stride);
+        const float f = ml.y > 0.0f ? ex2(ml.x - M) : 0.0f;
+        L += f * ml.y;
+        if (threadIdx.x < 32) weight[s] = f;
+    }
+    L = warp_sum_f(L);
     __syncthreads();
-    for (int s = 0; s < p.splits; ++s) L += weight[s] * w[s * stride + 1];
     if (p.sink) L += ex2(sk - M);
     float g = L > 0.0f ? 1.0f / L : 0.0f;
     if (p.gate) g *= sigmoid_f(to_f32(((const __nv_bfloat16*)p.gate)[row * p.gate_stride + head]));
@@ -396,7 +436,8 @@ __global__ void __launch_bounds__(128) attn_shared_combine_kernel(const AttnPara
 
 static int shared_stages(const ktk_attn& a, int n) {
     const int kc = (a.dim_stride + 63) / 64, fixed = kc * n * 128 + kAsTok * 128;
-    const int fit = (kAsSmem - fixed) / (kc * kAsChunk);
+    int fit = (kAsSmem - fixed) / (kc * kAsChunk);
+    if (fit > kAsMaxBars / kc) fit = kAsMaxBars / kc;
     return fit < kAsMaxStages ? fit : kAsMaxStages;
 }
 
@@ -410,7 +451,16 @@ int32_t attn_shared_splits(const ktk_attn& a, int batch, int new_rows, int64_t m
     const Packing k = packing_of(a.heads, new_rows == 0);
     const int64_t units = (int64_t)batch * k.chunks * (new_rows == 0 ? 1 : (new_rows + k.rows - 1) / k.rows);
     const int64_t tiles = (max_keys + kAsTok - 1) / kAsTok;
-    return fill_rounds(units, sm_count(), 1, 4, (tiles + kAsMinTiles - 1) / kAsMinTiles, kAsMaxSplits);
+    // rounds of CTAs x (tiles of each + what starting and finishing one costs, in tiles)
+    int64_t most = (tiles + kAsMinTiles - 1) / kAsMinTiles, best = 1, best_cost = -1;
+    if (most > kAsMaxSplits) most = kAsMaxSplits;
+    for (int64_t s = 1; s <= most && units > 0; ++s) {
+        const int64_t rounds = (units * s + sm_count() - 1) / sm_count();
+        const int64_t cost = rounds * ((tiles + s - 1) / s + kAsStartTiles) + (s > 1 ? kAsStartTiles : 0);
+        if (best_cost < 0 || cost < best_cost) { best_cost = cost; best = s; }
+        if (rounds > 8) break;
+    }
+    return (int32_t)best;
 }
 
 size_t attn_shared_workspace(const ktk_attn& a, int64_t rows, int splits) {
