@@ -22,7 +22,7 @@ constexpr int kAsChunk = kAsTok * 128;        // [64 tokens][64 columns]
 constexpr int kAsMaxStages = 8, kAsMaxBars = 40;
 constexpr int kAsSmem = 232448 - 2048;        // for Q, the ring and P; static arrays and alignment aside
 constexpr int kAsMinTiles = 4;                // a split is not worth less
-constexpr int kAsMaxSplits = 256, kAsStartTiles = 2;
+constexpr int kAsMaxSplits = 256, kAsStartTiles = 5;
 constexpr int kAsMaxDim = 576, kAsMaxVdim = 512;
 constexpr float kAsSlack = 8.0f;
 constexpr float kAsNone = -1e30f;             // reference of a column without a sink
@@ -70,7 +70,7 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
                    const uint32_t tmem_cols) {
     extern __shared__ uint8_t as_raw[];
     // a stage has landed; a pair of its chunks has been read out
-    __shared__ __align__(8) uint64_t full[kAsMaxStages], free_[kAsMaxBars], bar_s[2], bar_p, bar_o;
+    __shared__ __align__(8) uint64_t full[kAsMaxStages], free_[kAsMaxBars], bar_s[2], bar_p, bar_o, bar_q;
     __shared__ __align__(16) float ref_s[N], alpha_s[N];
     __shared__ __align__(16) int vis_s[N];
     __shared__ uint32_t tmem_base_s;
@@ -91,6 +91,7 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
     const int first = (int)(blockIdx.z % groups) * pk.rows;          // the CTA's first row within the sequence
     if (first >= n_new) return;                         // uniform for the CTA: nothing allocated yet
     const int rows = n_new - first < pk.rows ? n_new - first : pk.rows;
+    const bool one = pk.rows == 1;
     const int head0 = blockIdx.y * pk.heads, heads = a.heads - head0 < pk.heads ? a.heads - head0 : pk.heads;
     const Span s = span_of(p.t, b);
     const int base = s.total - n_new;
@@ -108,30 +109,12 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
         for (int i = 0; i < stages * pairs; ++i) mbar_init(&free_[i], 1);
         mbar_init(&bar_s[0], 1); mbar_init(&bar_s[1], 1);
         mbar_init(&bar_p, 128);
+        mbar_init(&bar_q, 128);
         mbar_init(&bar_o, 1);
         abort_flag = 0;
         mbar_init_fence();
     }
-    // column c: row first + c / heads of the sequence, head head0 + c % heads
-    if (warp < 4) {
-        for (int c = tid; c < N; c += 128) {
-            const int lr = c / pk.heads, h = c - lr * pk.heads;
-            const bool on = lr < rows && h < heads;
-            ref_s[c] = on && p.sink ? p.sink[head0 + h] * kLog2eF : kAsNone;
-            vis_s[c] = on ? base + first + lr + 1 : 0;
-        }
-        for (int i = tid; i < N * kc * 8; i += 128) {
-            const int c = i / (kc * 8), piece = i - c * (kc * 8), lr = c / pk.heads, h = c - lr * pk.heads;
-            uint4 v = make_uint4(0u, 0u, 0u, 0u);
-            if (lr < rows && h < heads && piece * 8 < a.dim_stride)
-                v = __ldg(reinterpret_cast<const uint4*>((const __nv_bfloat16*)p.q + (int64_t)(r0 + first + lr) * p.q_stride +
-                                                         (int64_t)(head0 + h) * a.dim_stride) + piece);
-            *reinterpret_cast<uint4*>(sQ + (piece >> 3) * (N * 128) + swz(c, piece & 7)) = v;
-        }
-        fence_proxy_async();
-    } else if (issuer) {
-        tmem_alloc(&tmem_base_s, tmem_cols);
-    }
+    if (issuer) tmem_alloc(&tmem_base_s, tmem_cols);
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -145,7 +128,8 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
         int s_at = 0, o_at = 0;                          // next tile of each product
         int s_st = 0, o_st = 0;                          // their stages
         uint32_t s_par = 0, idle = 0;
-        while (o_at < n) {
+        const bool started = mbar_wait_all(&bar_q, 0, &abort_flag);
+        while (started && o_at < n) {
             uint32_t ready = 0;
             if (o_at < s_at && __all_sync(0xffffffffu, mbar_test(&bar_p, o_at & 1))) ready |= 1u;
             if (s_at < n && s_at <= o_at + ((ready & 1u) ? 2 : 1) && __all_sync(0xffffffffu, mbar_test(&full[s_st], s_par))) ready |= 2u;
@@ -240,6 +224,31 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
         }
     } else {
         const uint32_t my = tmem + ((uint32_t)(warp * 32) << 16);
+        // column c: row first + c / heads of the sequence, head head0 + c % heads.  Q comes while the first tiles are on their
+        // way: 8 threads take a column, 16 bytes of every chunk each
+        for (int c = tid; c < N; c += 128) {
+            const int lr = one ? 0 : c / pk.heads, h = c - lr * pk.heads;
+            const bool on = lr < rows && h < heads;
+            ref_s[c] = on && p.sink ? p.sink[head0 + h] * kLog2eF : kAsNone;
+            vis_s[c] = on ? base + first + lr + 1 : 0;
+        }
+        for (int c = tid >> 3; c < N; c += 16) {
+            const int lr = one ? 0 : c / pk.heads, h = c - lr * pk.heads;
+            const bool on = lr < rows && h < heads;
+            const uint4* src = reinterpret_cast<const uint4*>(
+                (const __nv_bfloat16*)p.q + (int64_t)(r0 + first + (on ? lr : 0)) * p.q_stride +
+                (int64_t)(head0 + (on ? h : 0)) * a.dim_stride) + (tid & 7);
+            uint4 v[kAsMaxDim / 64];
+#pragma unroll
+            for (int k = 0; k < kAsMaxDim / 64; ++k)
+                v[k] = on && k * 64 + (tid & 7) * 8 < a.dim_stride ? __ldg(src + k * 8) : make_uint4(0u, 0u, 0u, 0u);
+#pragma unroll
+            for (int k = 0; k < kAsMaxDim / 64; ++k)
+                if (k < kc) *reinterpret_cast<uint4*>(sQ + k * (N * 128) + swz(c, tid & 7)) = v[k];
+        }
+        fence_proxy_async();
+        mbar_arrive(&bar_q);
+        softmax_warps_sync();
         // a thread holds two tokens of the tile and, of every 8 columns, the two from 2 (lane % 4) on
         const int tok = warp * 16 + (lane >> 2), col = 2 * (lane & 3);
         const float f = a.scale * kLog2eF;
@@ -342,7 +351,7 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
         softmax_warps_sync();
         for (int c = tid; c < N; c += 128) {
             float L = scratch[c] + scratch[N + c] + scratch[2 * N + c] + scratch[3 * N + c];
-            const int lr = c / pk.heads, h = head0 + c - lr * pk.heads;
+            const int lr = one ? 0 : c / pk.heads, h = head0 + c - lr * pk.heads;
             if (c - lr * pk.heads < heads && lr < rows) {
                 const int64_t row = r0 + first + lr;
                 if (p.splits > 1) {
@@ -366,7 +375,7 @@ attn_shared_kernel(const AttnParams p, const __grid_constant__ CUtensorMap k_map
 #pragma unroll
                 for (int c = 0; c < N; ++c) {
                     if (col >= a.vdim_stride) break;
-                    const int lr = c / pk.heads, h = head0 + c - lr * pk.heads;
+                    const int lr = one ? 0 : c / pk.heads, h = head0 + c - lr * pk.heads;
                     if (c - lr * pk.heads >= heads || lr >= rows) continue;
                     const int64_t row = r0 + first + lr;
                     if (p.splits > 1)

@@ -26,6 +26,12 @@ from .engine import PooledTable
 EXPAND_ROWS = 64        # from this many new tokens on, keys and values are expanded from the latents
 
 
+def _rounded_up(n: int) -> int:
+    """n to four leading bits, upwards: lengths that grow token by token change a launch's shape rarely."""
+    step = 1 << max(n.bit_length() - 4, 0)
+    return (n + step - 1) // step * step
+
+
 @dataclass
 class LatentWeights:
     """What a latent-attention layer brings to the manager: expansions of the latent to every head's keys
@@ -121,7 +127,7 @@ class LayeredKVManager(PooledTable):
         return LayerStep(table, new_indptr, slots_dev, len(slots), int(self._host_len[layer_idx][slots].max()))
 
     def _attention(self, q, k, v, step: LayerStep, spec: layer_ops.AttentionSpec, seq_len: int, **kw) -> torch.Tensor:
-        splits = layer_ops.attention_splits(spec, step.sequences, 1 << (step.longest - 1).bit_length(), self.dtype,
+        splits = layer_ops.attention_splits(spec, step.sequences, _rounded_up(step.longest), self.dtype,
                                             0 if step.new_indptr is None else seq_len)
         need = layer_ops.attention_workspace(spec, q.shape[0], splits, self.dtype)
         if need and (self._workspace is None or self._workspace.numel() < need):
