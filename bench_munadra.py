@@ -26,7 +26,7 @@ VOCAB, DIM, ROT, VDIM, RANK, TAPS, DENSE = 32768, 128, 64, 128, 512, 4, 3
 LIKE = {"attention": "attention", "append": "append", "row_norms": "row_norms", "router": "router",
         "experts_gate_up": "experts_gate_up", "experts_down": "experts_down", "projection_latent": "projection",
         "projection_lru": "projection", "expand_latents": "projection", "gather_latents": "append", "query_expansion": "projection",
-        "value_expansion": "projection", "lru_gate_products": "projection", "lru_conv": "row_norms", "lru_scan": "row_norms",
+        "value_expansion": "projection", "lru_gate_products": "projection", "lru_conv": "row_norms", "lru_scan": "row_norms", "lru_step": "row_norms",
         "dense_gate_up": "projection", "dense_activation": "row_norms", "output_projection": "projection"}
 
 
@@ -193,17 +193,21 @@ def _kernels(args, models, rec, lat, n, B, ctx, dev, timer, hbm, mm):
         proj, slots = rnd(rows, 2 * W), torch.arange(batch, dtype=torch.int32, device=dev)
         state, ring = torch.zeros(batch, W, device=dev), torch.zeros(batch, rec.taps, W, dtype=torch.bfloat16, device=dev)
         kw = dict(new_indptr=indptr, max_new=new)
-        per_step = 0 if prompt else rows * W
         gemm(ours, "projection_lru", h, LR["proj"], lambda: torch.addmm(LR["proj_b"], h, LR["proj"].t()))
-        record(ours, "lru_conv", lambda: lo.lru_conv(proj, rec, table, slots, w.conv_w, w.conv_b, ring, **kw), 0,
-               rows * W * 4 + per_step * rec.taps * 2)
-        u = rnd(rows, W)
-        record(ours, "lru_gate_products", lambda: lo.lru_gate_products(u, w.gates, rec), 4.0 * rows * W * W / rec.blocks,
-               rows * W * (2 + 8) + w.gates.numel() * 2)
-        zz = lo.lru_gate_products(u, w.gates, rec)
-        record(ours, "lru_scan", lambda: lo.lru_scan(zz, u, proj, rec, table, slots, w.rb, w.ib, w.decay, state, **kw), 0,
-               rows * W * (8 + 2 + 2 + 2) + per_step * 8)
-        del proj, u, zz
+        if prompt:
+            record(ours, "lru_conv", lambda: lo.lru_conv(proj, rec, table, slots, w.conv_w, w.conv_b, ring, **kw), 0,
+                   rows * W * 4)
+            u = rnd(rows, W)
+            record(ours, "lru_gate_products", lambda: lo.lru_gate_products(u, w.gates, rec), 4.0 * rows * W * W / rec.blocks,
+                   rows * W * (2 + 8) + w.gates.numel() * 2)
+            zz = lo.lru_gate_products(u, w.gates, rec)
+            record(ours, "lru_scan", lambda: lo.lru_scan(zz, u, proj, rec, table, slots, w.rb, w.ib, w.decay, state, **kw), 0,
+                   rows * W * (8 + 2 + 2 + 2))
+        else:
+            record(ours, "lru_step", lambda: lo.lru_decode(proj, rec, table, slots, w.conv_w, w.conv_b, w.gates, w.rb, w.ib, w.decay,
+                                                           ring, state), 4.0 * rows * W * W / rec.blocks,
+                   rows * W * (2 * (rec.taps + 1) + 2 + 2 + 8) + w.gates.numel() * 2)
+        del proj
 
         # ---- feed-forward
         record(ours, "row_norms", lambda: lo.residual_norm(x, h, C, 1e-6, y=y, post=LA["norm1"], center=False), 0, rows * C * 12)

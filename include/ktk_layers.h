@@ -160,6 +160,14 @@ KTK_API int ktk_lru_scan(const float* z, const void* u, const void* proj, int64_
                          int64_t num_slots, const float* rb, const float* ib, const float* decay, float* state,
                          void* out, const ktk_paged* table, const ktk_lru* shape, int32_t* status, void* stream);
 
+/* ktk_lru_conv, the gate products and ktk_lru_scan of one token of every sequence in one launch (bf16; blocks of channels
+ * up to what ktk_lru_decode_supported accepts).  gates [blocks, 2, block_stride, block_stride]: r's rows, then i's. */
+KTK_API int ktk_lru_decode_supported(const ktk_lru* shape);
+KTK_API int ktk_lru_decode(const void* proj, int64_t row_stride, int64_t y_col, int64_t x_col, int64_t rows,
+                           const int32_t* slots, int64_t num_slots, const float* conv_w, const float* conv_b,
+                           const void* gates, const float* rb, const float* ib, const float* decay, void* ring, float* state,
+                           void* out, const ktk_paged* table, const ktk_lru* shape, int32_t* status, void* stream);
+
 /* Mixture of experts over rows h [rows, width_stride]. */
 typedef struct ktk_moe {
     int32_t experts, top;

@@ -180,6 +180,10 @@ _LAYER_SIGNATURES = {
     "ktk_lru_scan": (c_int32, [c_void_p, c_void_p, c_void_p, c_int64, c_int64, _i32p, c_int64, c_int32, _i32p, c_int64,
                                c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, POINTER(Paged), POINTER(Lru), _i32p,
                                c_void_p]),
+    "ktk_lru_decode_supported": (c_int32, [POINTER(Lru)]),
+    "ktk_lru_decode": (c_int32, [c_void_p, c_int64, c_int64, c_int64, c_int64, _i32p, c_int64, c_void_p, c_void_p, c_void_p,
+                                 c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, POINTER(Paged), POINTER(Lru),
+                                 _i32p, c_void_p]),
     "ktk_gated_rows": (c_int32, [c_void_p, c_void_p, c_int64, c_int32, c_float, c_float, c_float, c_int32, c_void_p]),
     "ktk_scale_cap": (c_int32, [c_void_p, c_int64, c_float, c_float, c_void_p]),
     "ktk_moe_route": (c_int32, [c_void_p, c_void_p, c_void_p, _i32p, c_void_p, _i32p, _i32p, c_int64, POINTER(Moe),

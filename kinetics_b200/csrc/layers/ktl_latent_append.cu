@@ -7,20 +7,6 @@ namespace ktk {
 
 constexpr int kLaThreads = 128;
 
-template <typename T> struct Pair;
-template <> struct Pair<float> {
-    static __device__ __forceinline__ float2 load(const float* p) { return *reinterpret_cast<const float2*>(p); }
-    static __device__ __forceinline__ void store(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
-};
-template <> struct Pair<__nv_bfloat16> {
-    static __device__ __forceinline__ float2 load(const __nv_bfloat16* p) {
-        return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
-    }
-    static __device__ __forceinline__ void store(__nv_bfloat16* p, float a, float b) {
-        *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b);
-    }
-};
-
 template <typename T>
 __global__ void __launch_bounds__(kLaThreads)
 latent_append_kernel(T* proj, int64_t row_stride, int64_t q_col, int64_t kv_col, const int32_t* __restrict__ new_indptr,
@@ -37,25 +23,29 @@ latent_append_kernel(T* proj, int64_t row_stride, int64_t q_col, int64_t kv_col,
         if (tid == 0) report(status, KTK_STATUS_BAD_TABLE);
         return;
     }
-    const int half = a.rot_dim / 2, pairs = a.rot_stride / 2;
-    for (int i = tid; i < half; i += kLaThreads) {
-        float sn, cs;
-        sincosf((float)pos * freqs[i], &sn, &cs);
+    const int half = a.rot_dim / 2, vecs = a.rot_stride / 8;           // vecs: 8 columns, 4 pairs each
+    for (int i = tid; i < 4 * vecs; i += kLaThreads) {
+        float sn = 0.0f, cs = 0.0f;                       // behind the rotated columns: zeros
+        if (i < half) sincosf((float)pos * freqs[i], &sn, &cs);
         la_turn[i] = make_float2(cs * a.rot_factor, sn * a.rot_factor);
     }
     __syncthreads();
     const int head_cols = a.dim_stride + a.rot_stride, row_cols = a.rank_stride + a.rot_stride;
     T* row = proj + r * row_stride;
     auto turn = [&](const T* src, T* dst, int i) {
-        float2 v = make_float2(0.0f, 0.0f);
-        if (i < half) {
-            const float2 uv = Pair<T>::load(src + 2 * i), cs = la_turn[i];
-            v = make_float2(uv.x * cs.x - uv.y * cs.y, uv.y * cs.x + uv.x * cs.y);
+        float v[8];
+        Vec8<T>::load(src + 8 * i, v);
+#pragma unroll
+        for (int e = 0; e < 8; e += 2) {
+            const float2 cs = la_turn[4 * i + e / 2];
+            const float x = v[e], y = v[e + 1];
+            v[e] = x * cs.x - y * cs.y;
+            v[e + 1] = y * cs.x + x * cs.y;
         }
-        Pair<T>::store(dst + 2 * i, v.x, v.y);
+        Vec8<T>::store(dst + 8 * i, v);
     };
-    for (int j = tid; j < a.heads * pairs; j += kLaThreads) {
-        const int h = j / pairs, i = j - h * pairs;
+    for (int j = tid; j < a.heads * vecs; j += kLaThreads) {
+        const int h = j / vecs, i = j - h * vecs;
         T* src = row + q_col + (int64_t)h * head_cols + a.dim_stride;
         turn(src, q_out ? q_out + (r * a.heads + h) * row_cols + a.rank_stride : src, i);
     }
@@ -67,7 +57,7 @@ latent_append_kernel(T* proj, int64_t row_stride, int64_t q_col, int64_t kv_col,
     }
     const T* kv = row + kv_col;
     T* dst = pages + (page * t.page_size + pos % t.page_size) * row_cols;
-    for (int i = tid; i < pairs; i += kLaThreads) turn(kv + a.rank_stride, dst + a.rank_stride, i);
+    for (int i = tid; i < vecs; i += kLaThreads) turn(kv + a.rank_stride, dst + a.rank_stride, i);
     float ss = 0.0f;
     for (int c = tid * 8; c < a.rank_stride; c += kLaThreads * 8) {
         float v[8];

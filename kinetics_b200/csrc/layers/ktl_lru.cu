@@ -59,6 +59,7 @@ lru_conv_kernel(const T* __restrict__ x, int64_t row_stride, const int32_t* __re
             load8(w + (int64_t)k * width + c, wt[k]);
             if (k + 1 < TAPS) input(t0 - (TAPS - 1) + k, win[k]);
         }
+#pragma unroll 4
         for (int i = t0; i < t1; ++i) {
             input(i, win[TAPS > 0 ? TAPS - 1 : 0]);
             float o[8];
@@ -251,6 +252,151 @@ __global__ void __launch_bounds__(kLdThreads) lru_step_kernel(const LruParams p)
     ((T*)p.out)[r.row0 * width + c] = from_f32<T>(S * gelu_tanh<FAST>(to_f32(((const T*)p.y)[r.row0 * p.row_stride + c])));
 }
 
+// ---- one token of every sequence in one launch: convolution, gate products on the tensor cores, recurrence, output gate ----
+// A CTA takes 32 channels of a block and up to 32 rows.  It convolves all channels of the block (the products need them;
+// their inputs lie in L2), multiplies u [32 x block] with the 32 + 32 gate rows by mma.m16n8k16, and finishes its channels.
+// The ring's place that a step writes is read by no other CTA.
+constexpr int kLfRows = 32, kLfChan = 32, kLfThreads = 256, kLfMaxBlock = 512;
+
+__host__ __device__ inline int lf_ld(int block_stride) { return (block_stride + 15) / 16 * 16 + 8; }      // padded: no bank conflicts
+__host__ __device__ inline int lf_smem(int block_stride) { return (kLfRows + 2 * kLfChan) * lf_ld(block_stride) * 2 + kLfRows * (2 * kLfChan + 1) * 4; }
+
+struct LruDecodeParams {
+    LruParams p;
+    const __nv_bfloat16 *x, *gates;
+    const float *conv_w, *conv_b;
+    __nv_bfloat16* ring;
+};
+
+template <int TAPS> __global__ void __launch_bounds__(kLfThreads) lru_decode_kernel(const LruDecodeParams q) {
+    extern __shared__ __align__(16) uint8_t lf_raw[];
+    __shared__ int row_slot[kLfRows], row_pos[kLfRows];
+    const LruParams& p = q.p;
+    const int bs = p.a.block_stride, taps = p.a.taps, width = p.a.blocks * bs, ld = lf_ld(bs);
+    __nv_bfloat16* su = reinterpret_cast<__nv_bfloat16*>(lf_raw);       // [rows][ld]
+    __nv_bfloat16* sw = su + kLfRows * ld;                              // [32 rows of r, 32 of i][ld]
+    float* sz = reinterpret_cast<float*>(sw + 2 * kLfChan * ld);            // [rows][32 zr | 32 zi | pad]
+    constexpr int kZ = 2 * kLfChan + 1;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int slices = (bs + kLfChan - 1) / kLfChan, blk = blockIdx.x / slices, n0 = (blockIdx.x - blk * slices) * kLfChan;
+    const int64_t r0 = (int64_t)blockIdx.y * kLfRows;
+    const int rows = p.rows - r0 < kLfRows ? (int)(p.rows - r0) : kLfRows;
+    const int c0 = blk * bs, pieces = (ld - 8) / 8;                     // 16-byte pieces of a row
+    // gate weights on their way; rows and columns outside are zero
+    for (int i = tid; i < 2 * kLfChan * pieces; i += kLfThreads) {
+        const int n = i / pieces, k = i - n * pieces, c = n0 + (n & (kLfChan - 1));
+        const bool on = c < bs && k * 8 < bs;
+        const __nv_bfloat16* src = q.gates + (on ? ((int64_t)(2 * blk + n / kLfChan) * bs + c) * bs + k * 8 : 0);
+        asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(sw + n * ld + k * 8)), "l"(src),
+                     "r"(on ? 16u : 0u) : "memory");
+    }
+    if (tid < kLfRows) {
+        int slot = -1, pos = 0;
+        if (tid < rows) {
+            const Span s = span_of(p.t, (int)(r0 + tid));
+            slot = p.slots[r0 + tid];
+            pos = s.total - 1;
+            if (s.bad || pos < 0 || slot < 0 || slot >= p.num_slots) {
+                report(p.status, KTK_STATUS_BAD_TABLE);
+                slot = -1;
+            }
+        }
+        row_slot[tid] = slot;
+        row_pos[tid] = pos;
+    }
+    __syncthreads();
+    // u of every channel of the block: kBatch pieces per thread with all their loads in flight
+    constexpr int kBatch = TAPS > 0 ? 4 : 1, kTaps = TAPS > 0 ? TAPS : 1;
+    for (int i0 = tid; i0 < kLfRows * pieces; i0 += kLfThreads * kBatch) {
+        uint4 raw[kBatch][kTaps];
+#pragma unroll
+        for (int b = 0; b < kBatch; ++b) {
+            const int i = i0 + b * kLfThreads, r = i / pieces, k = i - r * pieces;
+            const bool on = i < kLfRows * pieces && row_slot[r & (kLfRows - 1)] >= 0 && k * 8 < bs;
+            const int slot = on ? row_slot[r] : 0, pos = on ? row_pos[r] : 0, c = c0 + k * 8;
+            const __nv_bfloat16* mine = q.ring + (int64_t)slot * taps * width + c;
+#pragma unroll
+            for (int t = 0; t < kTaps; ++t) {                           // the last is the token's own
+                const int at = pos - (kTaps - 1) + t;
+                raw[b][t] = make_uint4(0u, 0u, 0u, 0u);                 // zeros before the sequence
+                if (t == kTaps - 1) { if (on) raw[b][t] = *reinterpret_cast<const uint4*>(q.x + (r0 + r) * p.row_stride + c); }
+                else if (on && at >= 0) raw[b][t] = *reinterpret_cast<const uint4*>(mine + (int64_t)(at % taps) * width);
+            }
+        }
+#pragma unroll
+        for (int b = 0; b < kBatch; ++b) {
+            const int i = i0 + b * kLfThreads, r = i / pieces, k = i - r * pieces, c = c0 + k * 8;
+            if (i >= kLfRows * pieces) continue;
+            float o[8] = {0, 0, 0, 0, 0, 0, 0, 0};
+            if (row_slot[r] >= 0 && k * 8 < bs) {
+                __nv_bfloat16* mine = q.ring + (int64_t)row_slot[r] * taps * width + c;
+                float v[8], w[8];
+                load8(q.conv_b + c, o);
+                if (TAPS == 0)
+                    for (int t = 0; t + 1 < taps; ++t) {
+                        const int at = row_pos[r] - (taps - 1) + t;
+                        if (at < 0) continue;
+                        Vec8<__nv_bfloat16>::load(mine + (int64_t)(at % taps) * width, v);
+                        load8(q.conv_w + (int64_t)t * width + c, w);
+#pragma unroll
+                        for (int e = 0; e < 8; ++e) o[e] = fmaf(w[e], v[e], o[e]);
+                    }
+#pragma unroll
+                for (int t = 0; t < kTaps; ++t) {
+                    unpack8(raw[b][t], v);
+                    load8(q.conv_w + (int64_t)(taps - kTaps + t) * width + c, w);
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) o[e] = fmaf(w[e], v[e], o[e]);
+                }
+                if (k * 8 >= n0 && k * 8 < n0 + kLfChan)                 // this CTA's channels
+                    *reinterpret_cast<uint4*>(mine + (int64_t)(row_pos[r] % taps) * width) = raw[b][kTaps - 1];
+            }
+            Vec8<__nv_bfloat16>::store(su + r * ld + k * 8, o);
+        }
+    }
+    asm volatile("cp.async.wait_all;" ::: "memory");
+    __syncthreads();
+    {
+        // warp: 16 rows, 16 of the 64 columns
+        const int gid = lane >> 2, tig = lane & 3, m0 = (warp & 1) * 16, g0 = (warp >> 1) * 16;
+        float acc[2][4] = {};
+        const __nv_bfloat16* a0 = su + (m0 + gid) * ld + 2 * tig;
+        const __nv_bfloat16* b0 = sw + (g0 + gid) * ld + 2 * tig;
+#pragma unroll 4
+        for (int k = 0; k < ld - 8; k += 16) {
+            uint32_t a[4];
+            a[0] = *reinterpret_cast<const uint32_t*>(a0 + k);
+            a[1] = *reinterpret_cast<const uint32_t*>(a0 + 8 * ld + k);
+            a[2] = *reinterpret_cast<const uint32_t*>(a0 + k + 8);
+            a[3] = *reinterpret_cast<const uint32_t*>(a0 + 8 * ld + k + 8);
+#pragma unroll
+            for (int t = 0; t < 2; ++t)
+                mma_bf16(acc[t], a, *reinterpret_cast<const uint32_t*>(b0 + t * 8 * ld + k),
+                         *reinterpret_cast<const uint32_t*>(b0 + t * 8 * ld + k + 8));
+        }
+#pragma unroll
+        for (int t = 0; t < 2; ++t)
+#pragma unroll
+            for (int e = 0; e < 4; ++e) sz[(m0 + gid + (e >= 2 ? 8 : 0)) * kZ + g0 + t * 8 + 2 * tig + (e & 1)] = acc[t][e];
+    }
+    __syncthreads();
+    const int n = n0 + lane, c = c0 + n;
+    if (n >= bs) return;
+    const float rb = p.rb[c], ib = p.ib[c], decay = p.decay[c];
+#pragma unroll
+    for (int r = warp; r < kLfRows; r += kLfThreads / 32) {
+        const int slot = row_slot[r];
+        if (slot < 0) continue;
+        float* state = p.state + (int64_t)slot * width + c;
+        float a, g;
+        gates<true>(sz[r * kZ + lane], sz[r * kZ + kLfChan + lane], __bfloat162float(su[r * ld + n]), rb, ib, decay, a, g);
+        const float S = fmaf(a, row_pos[r] > 0 ? *state : 0.0f, g);
+        *state = S;
+        ((__nv_bfloat16*)p.out)[(r0 + r) * width + c] =
+            __float2bfloat16_rn(S * gelu_tanh<true>(__bfloat162float(((const __nv_bfloat16*)p.y)[(r0 + r) * p.row_stride + c])));
+    }
+}
+
 static int check_lru(const ktk_lru* a, const ktk_paged* t, const int32_t* new_indptr, int64_t rows, int32_t max_new,
                      int64_t row_stride, int64_t col, int64_t num_slots, const char* who) {
     if (a == nullptr || t == nullptr || a->blocks <= 0 || a->block <= 0 || a->block_stride < a->block ||
@@ -350,4 +496,36 @@ extern "C" int ktk_lru_scan(const float* z, const void* u, const void* proj, int
     const LruParams p{*shape, *table, z, u, (const char*)proj + y_col * size, row_stride, new_indptr, slots, num_slots, rows,
                       max_new, rb, ib, decay, state, out, status};
     return shape->dtype == KTK_F32 ? scan_launch<float>(p, (cudaStream_t)stream) : scan_launch<__nv_bfloat16>(p, (cudaStream_t)stream);
+}
+
+extern "C" int ktk_lru_decode_supported(const ktk_lru* shape) {
+    return shape && shape->dtype == KTK_BF16 && shape->block_stride > 0 && shape->block_stride <= kLfMaxBlock ? 1 : 0;
+}
+
+extern "C" int ktk_lru_decode(const void* proj, int64_t row_stride, int64_t y_col, int64_t x_col, int64_t rows,
+                              const int32_t* slots, int64_t num_slots, const float* conv_w, const float* conv_b,
+                              const void* gates, const float* rb, const float* ib, const float* decay, void* ring, float* state,
+                              void* out, const ktk_paged* table, const ktk_lru* shape, int32_t* status, void* stream) {
+    const char* who = "ktk_lru_decode";
+    int rc = check_lru(shape, table, nullptr, rows, 1, row_stride, x_col, num_slots, who);
+    if (rc == KTK_OK) rc = check_lru(shape, table, nullptr, rows, 1, row_stride, y_col, num_slots, who);
+    if (rc != KTK_OK) return rc;
+    if (!ktk_lru_decode_supported(shape)) { set_error("%s: bf16, blocks of at most %d channels", who, kLfMaxBlock); return KTK_ERR_UNSUPPORTED; }
+    if (rows == 0) return KTK_OK;
+    if (!proj || !slots || !conv_w || !conv_b || !gates || !rb || !ib || !decay || !ring || !state || !out || !table->kv_indptr ||
+        !table->kv_last_page_len ||
+        (((uintptr_t)proj | (uintptr_t)conv_w | (uintptr_t)conv_b | (uintptr_t)gates | (uintptr_t)ring) & 15u) != 0) {
+        set_error("%s: null or misaligned pointer", who);
+        return KTK_ERR_ARG;
+    }
+    const LruParams p{*shape, *table, nullptr, nullptr, (const __nv_bfloat16*)proj + y_col, row_stride, nullptr, slots, num_slots,
+                      rows, 1, rb, ib, decay, state, out, status};
+    const LruDecodeParams q{p, (const __nv_bfloat16*)proj + x_col, (const __nv_bfloat16*)gates, conv_w, conv_b, (__nv_bfloat16*)ring};
+    const int smem = lf_smem(shape->block_stride), slices = (shape->block_stride + kLfChan - 1) / kLfChan;
+    auto kernel = shape->taps == 4 ? lru_decode_kernel<4> : lru_decode_kernel<0>;
+    KTK_CUDA_TRY(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem), who);
+    kernel<<<dim3((unsigned)(shape->blocks * slices), (unsigned)((rows + kLfRows - 1) / kLfRows)), kLfThreads, smem,
+             (cudaStream_t)stream>>>(q);
+    KTK_CUDA_TRY(cudaGetLastError(), who);
+    return KTK_OK;
 }

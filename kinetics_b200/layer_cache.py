@@ -174,6 +174,9 @@ class LayeredKVManager(PooledTable):
     def recur(self, proj: torch.Tensor, layer_idx: int, batch_idx: torch.Tensor, seq_len: int, w: LruWeights) -> torch.Tensor:
         """proj [rows, y | x]: advances the slots' convolution and state, returns the gated state [rows, cols]."""
         spec, step = self.specs[layer_idx], self._step_of(layer_idx, batch_idx, seq_len)
+        if step.new_indptr is None and layer_ops.lru_decode_supported(spec, self.dtype):
+            return layer_ops.lru_decode(proj, spec, step.table, step.slots, w.conv_w, w.conv_b, w.gates, w.rb, w.ib, w.decay,
+                                        self.rings[layer_idx], self.states[layer_idx], status=self.status)
         run = dict(new_indptr=step.new_indptr, max_new=seq_len, status=self.status)
         u = layer_ops.lru_conv(proj, spec, step.table, step.slots, w.conv_w, w.conv_b, self.rings[layer_idx], **run)
         z = layer_ops.lru_gate_products(u, w.gates, spec)

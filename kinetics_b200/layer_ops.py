@@ -472,3 +472,29 @@ def lru_scan(z, u, proj, spec: LruSpec, table: PageTable, slots, rb, ib, decay, 
         _ptr(rb), _ptr(ib), _ptr(decay), _ptr(state), _ptr(out), ctypes.byref(t), ctypes.byref(a), _ptr(status), _stream()))
     _launched()
     return out
+
+
+def lru_decode_supported(spec: LruSpec, dtype) -> bool:
+    a = spec.c(_lib.KTK_BF16 if dtype == torch.bfloat16 else _lib.KTK_F32)
+    return bool(_lib.load_layers().ktk_lru_decode_supported(ctypes.byref(a)))
+
+
+def lru_decode(proj, spec: LruSpec, table: PageTable, slots, conv_w, conv_b, gates, rb, ib, decay, ring, state, status=None):
+    """lru_conv, lru_gate_products and lru_scan of one token of every sequence, in one launch (bf16)."""
+    _cuda(proj, slots, conv_w, conv_b, gates, rb, ib, decay, ring, state, status)
+    n = pad8(spec.block)
+    if proj.shape != (table.batch, 2 * spec.cols) or tuple(ring.shape[1:]) != (spec.taps, spec.cols) or \
+            tuple(gates.shape) != (spec.blocks, 2 * n, n) or tuple(conv_w.shape) != (spec.taps, spec.cols) or \
+            any(v.dtype != torch.float32 or v.numel() != spec.cols for v in (conv_b, rb, ib, decay)) or \
+            any(v.dtype != torch.bfloat16 for v in (proj, ring, gates)) or conv_w.dtype != torch.float32 or \
+            state.dtype != torch.float32 or state.shape != (ring.shape[0], spec.cols) or \
+            slots.dtype != torch.int32 or slots.numel() != table.batch:
+        raise ValueError(f"lru_decode: shapes {tuple(proj.shape)}, {tuple(ring.shape)} do not fit {spec}")
+    out = torch.empty(proj.shape[0], spec.cols, dtype=proj.dtype, device=proj.device)
+    a, t = spec.c(_lib.KTK_BF16), table.c()
+    check_layers(_lib.load_layers().ktk_lru_decode(
+        _ptr(proj), proj.shape[1], 0, spec.cols, proj.shape[0], _ptr(slots), ring.shape[0], _ptr(conv_w), _ptr(conv_b),
+        _ptr(gates), _ptr(rb), _ptr(ib), _ptr(decay), _ptr(ring), _ptr(state), _ptr(out), ctypes.byref(t), ctypes.byref(a),
+        _ptr(status), _stream()))
+    _launched()
+    return out

@@ -127,6 +127,8 @@ class Munadra(LayeredModel):
             layer.update(mixer(pack, p + "mix.", l.mixer))
             if l.ff:
                 layer.update(norm2=norm(p + "norm2"))
+            elif p + "norm2" in weights:                 # nothing to normalise
+                pack[p + "norm2"]
             if l.experts:
                 layer.update(pack.experts(p + "mlp.", layer["moe"], bias=False))
             elif l.ff:

@@ -225,12 +225,17 @@ class _Lru:
         self.state = torch.full((slots, spec.cols), float("nan"), device=dev)       # a new sequence reads none of it
         self.ring = torch.full((slots, spec.taps, spec.cols), float("nan"), device=dev, dtype=dtype)
 
-    def run(self, y, x, table, slots, new=None):
+    def run(self, y, x, table, slots, new=None, fused=False):
         from kinetics_b200 import layer_ops as lo, ops
         proj = torch.cat((y, x), dim=1).to(self.dtype).to(self.dev)
         status, slots = ops.new_status(self.dev), torch.tensor(slots, dtype=torch.int32, device=self.dev)
         kw = dict(new_indptr=None if new is None else torch.tensor([0, new], dtype=torch.int32, device=self.dev),
                   max_new=new or 1, status=status)
+        if fused and new is None and lo.lru_decode_supported(self.spec, self.dtype):
+            out = lo.lru_decode(proj, self.spec, table, slots, self.w, self.b, self.gates, self.rb, self.ib, self.decay,
+                                self.ring, self.state, status)
+            ops.raise_on_status(status)
+            return out.double().cpu()
         u = lo.lru_conv(proj, self.spec, table, slots, self.w, self.b, self.ring, **kw)
         z = lo.lru_gate_products(u, self.gates, self.spec)
         out = lo.lru_scan(z, u, proj, self.spec, table, slots, self.rb, self.ib, self.decay, self.state, **kw)
@@ -246,27 +251,28 @@ def _length_table(lens, dev, ps=16):
     return PageTable(i32(list(range(sum(pages)))), i32(indptr), i32([n - (c - 1) * ps for n, c in zip(lens, pages)]), ps, sum(pages))
 
 
+@pytest.mark.parametrize("fused", [False, True])
 @pytest.mark.parametrize("dtype", [F32, BF])
-@pytest.mark.parametrize("blocks,block,taps", [(3, 20, 4), (1, 48, 2), (2, 17, 1), (4, 8, 7), (2, 80, 4), (1, 16, 30)])
-def test_recurrence_in_portions(cuda_device, dtype, blocks, block, taps):
+@pytest.mark.parametrize("blocks,block,taps", [(1, 264, 4), (3, 20, 4), (1, 48, 2), (2, 17, 1), (4, 8, 7), (2, 80, 4), (1, 16, 30)])
+def test_recurrence_in_portions(cuda_device, dtype, blocks, block, taps, fused):
     from kinetics_b200.layer_ops import LruSpec
     spec = LruSpec(blocks, block, taps)
     total = 300
     c, spread = _lru_case(spec, total, blocks + taps)
     want = spread(_lru_plain(c, dtype).float()).double()
     y, x = spread(c["y"]), spread(c["x"])
-    lru = _Lru(spec, [c], spread, dtype, cuda_device, 3)
-    for slot, sizes in enumerate([[300], [2] * 150, [127, 1, 2, 129, 3, 16, 22]]):
+    lru = _Lru(spec, [c], spread, dtype, cuda_device, 4)
+    for slot, sizes in enumerate([[300], [2] * 150, [127, 1, 2, 129, 1, 1, 1, 16, 22], [1] * 300]):
         got, at = [], 0
         for n in sizes:
-            got.append(lru.run(y[at:at + n], x[at:at + n], _length_table([at + n], cuda_device), [slot], n if n > 1 else None))
+            got.append(lru.run(y[at:at + n], x[at:at + n], _length_table([at + n], cuda_device), [slot], n if n > 1 else None, fused))
             at += n
         err = (torch.cat(got) - want).pow(2).mean(-1).sqrt() / rms(want)
         assert err.max() < (2e-5 if dtype == F32 else 2e-2), (sizes, float(err.max()))
 
 
-@pytest.mark.parametrize("dtype", [F32, BF])
-def test_recurrence_of_unequal_sequences(cuda_device, dtype):
+@pytest.mark.parametrize("dtype,fused", [(F32, False), (BF, False), (BF, True)])
+def test_recurrence_of_unequal_sequences(cuda_device, dtype, fused):
     # prompts of different lengths, then steps of all of them together in changing order; then a slot is used again
     from kinetics_b200.layer_ops import LruSpec
     spec, lens, steps = LruSpec(2, 24, 4), [1, 2, 5, 70], 40
@@ -287,7 +293,8 @@ def test_recurrence_of_unequal_sequences(cuda_device, dtype):
     for t in range(steps):
         order = [(k + t) % 4 for k in range(4)]
         rows = lambda key: torch.cat([spread(cases[i][key][lens[i] + t:lens[i] + t + 1]) for i in order])
-        out = lru.run(rows("y"), rows("x"), _length_table([lens[i] + t + 1 for i in order], cuda_device), [slot_of[i] for i in order])
+        out = lru.run(rows("y"), rows("x"), _length_table([lens[i] + t + 1 for i in order], cuda_device), [slot_of[i] for i in order],
+                      None, fused)
         for k, i in enumerate(order):
             got[i].append(out[k:k + 1])
     prompt(4, 30, slot_of[3])
@@ -296,6 +303,29 @@ def test_recurrence_of_unequal_sequences(cuda_device, dtype):
         mine = torch.cat(got[i])
         err = (mine - want[:mine.shape[0]]).pow(2).mean(-1).sqrt() / rms(want)
         assert err.max() < (2e-5 if dtype == F32 else 2e-2), (i, float(err.max()))
+
+
+def test_fused_steps_of_many_sequences_equal_the_separate_ones(cuda_device):
+    # more rows than a CTA takes, in permuted slots; some start now
+    from kinetics_b200.layer_ops import LruSpec
+    dev, g = cuda_device, torch.Generator().manual_seed(0)
+    for spec in (LruSpec(2, 40, 4), LruSpec(1, 512, 3), LruSpec(3, 33, 2)):
+        rows = 150
+        c, spread = _lru_case(spec, rows, 4)
+        a, b = (_Lru(spec, [c], spread, BF, dev, rows + 7) for _ in range(2))
+        slots = torch.randperm(rows + 7, generator=g)[:rows].tolist()
+        for lru in (a, b):
+            h = torch.Generator().manual_seed(1)
+            lru.state.copy_(torch.randn(lru.state.shape, generator=h))
+            lru.ring.copy_(torch.randn(lru.ring.shape, generator=h))
+        lens = torch.randint(1, 60, (rows,), generator=g).tolist()
+        lens[:5] = [1, 2, 3, 4, 5]
+        for step in range(3):
+            table = _length_table([n + step for n in lens], dev)
+            one, two = (m.run(spread(c["y"]), spread(c["x"]), table, slots, None, f) for m, f in ((a, False), (b, True)))
+            torch.testing.assert_close(one, two, rtol=2e-2, atol=2e-3)
+        torch.testing.assert_close(a.state, b.state, rtol=1e-3, atol=1e-4)
+        assert torch.equal(a.ring, b.ring)
 
 
 @pytest.mark.parametrize("dtype", [F32, BF])
