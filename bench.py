@@ -112,7 +112,8 @@ def parse():
                     help="time one kernel alone on the workload's shapes (select: only the page summaries are "
                          "allocated, so the full batch fits in a few GB; exchange: the NVLink exchange kernels "
                          "on [batch, hidden] under torchrun, every form, beside NCCL; gifetar: prefill and decode of "
-                         "Gifetar layers, kernel by kernel, beside DecoderStack at equal size)")
+                         "Gifetar layers, kernel by kernel, beside DecoderStack at equal size; munadra: the same of Munadra "
+                         "layers beside Gifetar)")
     ap.add_argument("--only-kernel", default="", help="--micro gifetar, munadra: time only the kernels whose name holds this")
     return ap.parse_args()
 
