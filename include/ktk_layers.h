@@ -111,13 +111,13 @@ typedef struct ktk_latent {
 /*
  * One launch per layer over rows of proj [rows, row_stride]:
  *   queries at q_col: heads of [dim_stride | rot_stride]; the rotated part (pairs 2 i, 2 i + 1 turned by position *
- *   freqs[i], fp32 [rot_dim / 2]) goes to q_out [rows, heads, rank_stride + rot_stride], columns rank_stride.., or back
+ *   turns[i] whole turns, fp64 [rot_dim / 2]) goes to q_out [rows, heads, rank_stride + rot_stride], columns rank_stride.., or back
  *   in place where q_out is null;
  *   latents at kv_col (< 0: none): [rank_stride | rot_stride]; norm(latent) * norm_w (fp32 [rank_stride]) and the
  *   rotated key go to the token's page row.
  */
 KTK_API int ktk_latent_append(void* proj, int64_t row_stride, int64_t q_col, int64_t kv_col, const int32_t* new_indptr,
-                              int64_t rows, const float* norm_w, const float* freqs, void* q_out, void* pages,
+                              int64_t rows, const float* norm_w, const double* turns, void* q_out, void* pages,
                               const ktk_paged* table, const ktk_latent* shape, int32_t* status, void* stream);
 
 /*

@@ -10,7 +10,7 @@ constexpr int kLaThreads = 128;
 template <typename T>
 __global__ void __launch_bounds__(kLaThreads)
 latent_append_kernel(T* proj, int64_t row_stride, int64_t q_col, int64_t kv_col, const int32_t* __restrict__ new_indptr,
-                     const float* __restrict__ norm_w, const float* __restrict__ freqs, T* q_out, T* pages,
+                     const float* __restrict__ norm_w, const double* __restrict__ turns, T* q_out, T* pages,
                      const ktk_paged t, const ktk_latent a, int32_t* status) {
     extern __shared__ float2 la_turn[];                   // cos, sin of every pair
     __shared__ float part[kLaThreads / 32];
@@ -26,7 +26,11 @@ latent_append_kernel(T* proj, int64_t row_stride, int64_t q_col, int64_t kv_col,
     const int half = a.rot_dim / 2, vecs = a.rot_stride / 8;           // vecs: 8 columns, 4 pairs each
     for (int i = tid; i < 4 * vecs; i += kLaThreads) {
         float sn = 0.0f, cs = 0.0f;                       // behind the rotated columns: zeros
-        if (i < half) sincosf((float)pos * freqs[i], &sn, &cs);
+        if (i < half) {
+            // the whole turns are taken off before rounding: far positions keep their angle
+            const double whole = (double)pos * turns[i];
+            sincospif((float)(2.0 * (whole - rint(whole))), &sn, &cs);
+        }
         la_turn[i] = make_float2(cs * a.rot_factor, sn * a.rot_factor);
     }
     __syncthreads();
@@ -84,7 +88,7 @@ latent_append_kernel(T* proj, int64_t row_stride, int64_t q_col, int64_t kv_col,
 using namespace ktk;
 
 extern "C" int ktk_latent_append(void* proj, int64_t row_stride, int64_t q_col, int64_t kv_col, const int32_t* new_indptr,
-                                 int64_t rows, const float* norm_w, const float* freqs, void* q_out, void* pages,
+                                 int64_t rows, const float* norm_w, const double* turns, void* q_out, void* pages,
                                  const ktk_paged* table, const ktk_latent* shape, int32_t* status, void* stream) {
     const char* who = "ktk_latent_append";
     int rc = check_latent(shape, who);
@@ -99,7 +103,7 @@ extern "C" int ktk_latent_append(void* proj, int64_t row_stride, int64_t q_col, 
     if (rows == 0) return KTK_OK;
     const int64_t q_cols = (int64_t)shape->heads * (shape->dim_stride + shape->rot_stride);
     const int kv_cols = shape->rank_stride + shape->rot_stride;
-    if (!proj || !freqs || !table->kv_indices || !table->kv_indptr || !table->kv_last_page_len || row_stride % 8 != 0 ||
+    if (!proj || !turns || !table->kv_indices || !table->kv_indptr || !table->kv_last_page_len || row_stride % 8 != 0 ||
         q_col % 8 != 0 || q_col < 0 || q_col + q_cols > row_stride ||
         (kv_col >= 0 && (kv_col % 8 != 0 || kv_col + kv_cols > row_stride || !norm_w || !pages)) ||
         (((uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)pages | (uintptr_t)norm_w) & 15u) != 0) {
@@ -110,11 +114,11 @@ extern "C" int ktk_latent_append(void* proj, int64_t row_stride, int64_t q_col, 
     cudaStream_t st = (cudaStream_t)stream;
     if (shape->dtype == KTK_F32)
         latent_append_kernel<float><<<(unsigned)rows, kLaThreads, smem, st>>>(
-            (float*)proj, row_stride, q_col, kv_col, new_indptr, norm_w, freqs, (float*)q_out, (float*)pages, *table, *shape,
+            (float*)proj, row_stride, q_col, kv_col, new_indptr, norm_w, turns, (float*)q_out, (float*)pages, *table, *shape,
             status);
     else
         latent_append_kernel<__nv_bfloat16><<<(unsigned)rows, kLaThreads, smem, st>>>(
-            (__nv_bfloat16*)proj, row_stride, q_col, kv_col, new_indptr, norm_w, freqs, (__nv_bfloat16*)q_out,
+            (__nv_bfloat16*)proj, row_stride, q_col, kv_col, new_indptr, norm_w, turns, (__nv_bfloat16*)q_out,
             (__nv_bfloat16*)pages, *table, *shape, status);
     KTK_CUDA_TRY(cudaGetLastError(), who);
     return KTK_OK;

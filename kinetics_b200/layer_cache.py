@@ -36,13 +36,13 @@ def _rounded_up(n: int) -> int:
 class LatentWeights:
     """What a latent-attention layer brings to the manager: expansions of the latent to every head's keys
     uk [heads, dim, rank] and values uv [heads, vdim, rank] (padded sizes; both views of ukv [heads * (dim + vdim), rank]),
-    sinks fp32 [heads], the latent's norm fp32 [rank] (None with kv_from), rotation frequencies fp32 [rot_dim / 2]."""
+    sinks fp32 [heads], the latent's norm fp32 [rank] (None with kv_from), turns per position fp64 [rot_dim / 2]."""
     ukv: torch.Tensor
     uk: torch.Tensor
     uv: torch.Tensor
     sink: torch.Tensor
     norm: Optional[torch.Tensor]
-    freqs: torch.Tensor
+    turns: torch.Tensor
 
 
 @dataclass
@@ -158,12 +158,12 @@ class LayeredKVManager(PooledTable):
         gate = proj[:, spec.gate_col:]
         dim, rank, vdim = w.uk.shape[1], w.uk.shape[2], w.uv.shape[1]
         if rows >= EXPAND_ROWS and step.new_indptr is not None and layer_ops.expanded_supported(spec, self.dtype):
-            layer_ops.latent_append(proj, spec, step.table, pages, w.norm, w.freqs, step.new_indptr, status=self.status)
+            layer_ops.latent_append(proj, spec, step.table, pages, w.norm, w.turns, step.new_indptr, status=self.status)
             latents = layer_ops.gather_rows(pages, step.table, step.longest, status=self.status)
             kv = torch.mm(latents[:, :rank], w.ukv.t())
             return layer_ops.expanded_attention(proj, kv, latents, spec, w.sink, gate, status=self.status)
         q = torch.empty(rows, H, spec.row_cols, dtype=proj.dtype, device=proj.device)
-        layer_ops.latent_append(proj, spec, step.table, pages, w.norm, w.freqs, step.new_indptr, q, status=self.status)
+        layer_ops.latent_append(proj, spec, step.table, pages, w.norm, w.turns, step.new_indptr, q, status=self.status)
         heads = proj[:, :spec.q_cols].view(rows, H, -1)
         torch.bmm(heads[:, :, :dim].transpose(0, 1), w.uk, out=q[:, :, :rank].transpose(0, 1))
         latent = self._attention(q.view(rows, -1), pages, pages, step, spec.rows(), seq_len, sink=w.sink, gate=gate)

@@ -119,7 +119,7 @@ class Rotation:
     scaled: bool = False
 
     def frequencies(self) -> torch.Tensor:
-        """fp32 [dims / 2]."""
+        """Radians per position, fp64 [dims / 2]."""
         i = torch.arange(self.dims // 2, dtype=torch.float64)
         f = self.base ** (-2.0 * i / self.dims)
         if self.scaled:
@@ -128,7 +128,11 @@ class Rotation:
             hi = min(math.ceil(pair_of(self.slow)), self.dims - 1)
             stretched = ((i - lo) / max(hi - lo, 0.001)).clamp(0.0, 1.0)
             f = torch.lerp(f, f / self.factor, stretched)
-        return f.float()
+        return f
+
+    def turns(self) -> torch.Tensor:
+        """Whole turns per position, fp64 [dims / 2]: what latent_append takes."""
+        return self.frequencies() / (2 * math.pi)
 
     @property
     def amplitude(self) -> float:
@@ -372,15 +376,15 @@ def scale_cap(z, scale: float, cap: float):
     return z
 
 
-def latent_append(proj, spec: LatentSpec, table: PageTable, pages, norm_w, freqs, new_indptr=None, q_out=None,
+def latent_append(proj, spec: LatentSpec, table: PageTable, pages, norm_w, turns, new_indptr=None, q_out=None,
                   status=None) -> None:
     """Turns the queries' rotated parts (into q_out [rows, heads, row_cols], or in place) and, where the layer has its
     own, writes normalised latents and rotated keys to their page rows (the table already includes them)."""
-    _cuda(proj, pages, norm_w, freqs, new_indptr, q_out, status)
-    if proj.dtype != pages.dtype or q_out is not None and q_out.dtype != proj.dtype or freqs.dtype != torch.float32 or \
+    _cuda(proj, pages, norm_w, turns, new_indptr, q_out, status)
+    if proj.dtype != pages.dtype or q_out is not None and q_out.dtype != proj.dtype or turns.dtype != torch.float64 or \
             norm_w is not None and norm_w.dtype != torch.float32:
-        raise TypeError("latent_append: proj, q_out and the cache share a dtype; norm and frequencies are fp32")
-    if proj.shape[1] != spec.proj_cols or freqs.numel() != spec.rot_dim // 2 or \
+        raise TypeError("latent_append: proj, q_out and the cache share a dtype; the norm is fp32, turns fp64")
+    if proj.shape[1] != spec.proj_cols or turns.numel() != spec.rot_dim // 2 or \
             tuple(pages.shape) != (table.num_pages, 1, table.page_size, spec.row_cols) or \
             q_out is not None and tuple(q_out.shape) != (proj.shape[0], spec.heads, spec.row_cols):
         raise ValueError(f"latent_append: shapes {tuple(proj.shape)}, {tuple(pages.shape)} do not fit {spec}")
@@ -388,7 +392,7 @@ def latent_append(proj, spec: LatentSpec, table: PageTable, pages, norm_w, freqs
     a, t = spec.c(_dtype_code(proj)), table.c()
     check_layers(_lib.load_layers().ktk_latent_append(
         _ptr(proj), proj.shape[1], 0, spec.q_cols if own else -1, _ptr(new_indptr), proj.shape[0],
-        _ptr(norm_w if own else None), _ptr(freqs), _ptr(q_out), _ptr(pages), ctypes.byref(t), ctypes.byref(a), _ptr(status),
+        _ptr(norm_w if own else None), _ptr(turns), _ptr(q_out), _ptr(pages), ctypes.byref(t), ctypes.byref(a), _ptr(status),
         _stream()))
     _launched()
 

@@ -161,7 +161,7 @@ class Munadra(LayeredModel):
         sink = pack.vector(mx + "sink", 1, s.heads)[:s.heads].contiguous()
         w = LatentWeights(ukv=ukv, uk=ukv[:cut].view(s.heads, -1, pad8(s.rank)), uv=ukv[cut:].view(s.heads, -1, pad8(s.rank)),
                           sink=sink, norm=pack.vector(mx + "dkv.norm", 1, s.rank) if own else None,
-                          freqs=s.rotation.frequencies().to(self.device))
+                          turns=s.rotation.turns().to(self.device))
         return dict(proj=torch.cat(parts), proj_b=None, out=pack.matrix(mx + "o", C, (s.heads, s.vdim)), mix=w)
 
     def _lru(self, pack, mx, s: LruSpec) -> dict:
