@@ -106,7 +106,7 @@ class MoeSpec:
 
 @dataclass(frozen=True)
 class Rotation:
-    """Rotary positions on pairs (2 i, 2 i + 1) of `dims` columns: base^(-2 i / dims) turns per position, and with
+    """Rotary positions on pairs (2 i, 2 i + 1) of `dims` columns: base^(-2 i / dims) radians per position, and with
     factor != 1 their stretch for contexts beyond `original` (YaRN): pairs that turn at least `fast` times within
     `original` positions keep their frequency, those that turn less than `slow` times have it divided by factor, a ramp
     in between; cos and sin are multiplied by 0.1 ln(factor) + 1."""
